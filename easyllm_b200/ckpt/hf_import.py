@@ -58,9 +58,28 @@ _INTERNLM2_RULES = [
     (r"^model\.layers\.(\d+)\.attention_norm\.weight$", r"\1:input_layernorm.weight"),
     (r"^model\.layers\.(\d+)\.ffn_norm\.weight$", r"\1:post_attention_layernorm.weight"),
 ]
+# Pafodra: name inside a layer on disk -> name in the layer's module (experts and mixes are stacked afterwards)
+PAFODRA_NAMES = {f"norm1{d}": f"input_layernorm.{n}" for d, n in (("", "weight"), (".b", "bias"), (".alpha", "alpha"))}
+PAFODRA_NAMES.update({f"mix.{p}": f"mixer.{p}_proj.weight" for p in
+                      ("q", "k", "v", "o", "r", "g", "w1", "w2", "a1", "a2", "g1", "g2", "b")})
+PAFODRA_NAMES.update({f"mix.{p}": f"mixer.{p}" for p in ("sink", "w0", "u", "norm", "A_log", "dt_bias")})
+PAFODRA_NAMES.update({f"mix.{p}.conv": f"mixer.{p}_conv" for p in "qkv"})
+for _p in ("gate", "up", "down"):
+    PAFODRA_NAMES[f"mlp.{_p}"], PAFODRA_NAMES[f"mlp.{_p}.b"] = f"mlp.{_p}_proj.weight", f"mlp.{_p}_proj.bias"
+PAFODRA_NAMES.update({"mlp.router": "mlp.router.weight", "mlp.shared.up": "mlp.shared.up_proj.weight",
+                      "mlp.shared.down": "mlp.shared.down_proj.weight", "mlp.shared.sg": "mlp.shared_gate.weight"})
+_PAFODRA_RULES = [(rf"^l(\d+)\.{re.escape(k)}$", rf"\1:{v}") for k, v in PAFODRA_NAMES.items()] + [
+    (r"^l(\d+)\.mix\.mu\.([rkvgw])$", r"\1:mixer.mu.\2"),
+    (r"^l(\d+)\.mlp\.e(\d+)\.(up|down)$", r"\1:mlp.experts.\2.\3"),
+    (r"^embed$", "embed:word_embeddings.weight"),
+    (r"^head$", "head:word_embeddings.weight"),
+    (r"^final\.norm$", "norm:weight"),
+    (r"^final\.norm\.b$", "norm:bias"),
+    (r"^final\.norm\.alpha$", "norm:alpha"),
+]
 RULES = {"llama": _LLAMA_RULES, "llama_pack": _LLAMA_RULES, "qwen": _QWEN_RULES,
          "internlm2": _INTERNLM2_RULES, "internlm2_pack": _INTERNLM2_RULES, "baichuan": _LLAMA_RULES,
-         "internlm": _LLAMA_RULES}
+         "internlm": _LLAMA_RULES, "pafodra": _PAFODRA_RULES}
 
 
 def canonicalize(hf_state: Dict[str, torch.Tensor], pretrain_type: str, n_heads: int, n_kv_heads: int,

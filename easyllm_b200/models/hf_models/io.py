@@ -11,7 +11,8 @@ import torch
 from ...ckpt.hf_import import canonicalize
 
 _FAMILY_RULES = {"llama": "llama", "internlm": "llama", "baichuan": "baichuan", "baichuan2": "baichuan",
-                 "baichuan2-13b": "baichuan", "internlm2": "internlm2", "qwen": "qwen"}
+                 "baichuan2-13b": "baichuan", "internlm2": "internlm2", "qwen": "qwen", "pafodra": "pafodra"}
+_MIXES = "rkvgw"          # rows of TimeMix.mu
 
 
 def import_state(hf_state, arch):
@@ -23,12 +24,66 @@ def import_state(hf_state, arch):
             if slot == "embed":
                 out["model.embed_tokens.weight"] = t
             elif slot == "norm":
-                out["model.norm.weight"] = t
+                out[f"model.norm.{name}"] = t
             elif slot == "head":
                 out["lm_head.weight"] = t
             else:
                 out[f"model.layers.{slot}.{name}"] = t
+    return _stack_hybrid(out, arch) if arch.layers is not None else out
+
+
+def sizes_from_state(arch, raw):
+    """Sizes that only the tensors tell (ranks of the low-rank projections) → the arch's layer specs."""
+    from .modeling import weight_owner
+    for i, spec in enumerate(arch.layers or []):
+        n = f"l{weight_owner(arch.layers, i)}.mix"
+        if spec.type == "wkv":
+            spec.mixer["decay_rank"] = raw[n + ".w1"].shape[0]
+        elif spec.type == "channel_delta":
+            spec.mixer["decay_rank"], spec.mixer["gate_rank"] = raw[n + ".a1"].shape[0], raw[n + ".g1"].shape[0]
+
+
+def _stack_hybrid(sd, arch):
+    """Per-expert and per-mix tensors stacked as the modules hold them, and the tensors of a layer repeated under the
+    index of every layer that uses them (``nn.Module.state_dict`` lists a shared module at each of its places)."""
+    from .modeling import weight_owner
+    out = {}
+    for i, spec in enumerate(arch.layers):
+        src, dst = f"model.layers.{weight_owner(arch.layers, i)}.", f"model.layers.{i}."
+        mine = {k[len(src):]: v for k, v in sd.items() if k.startswith(src)}
+        if spec.type == "wkv":
+            mine["mixer.mu"] = torch.stack([mine.pop(f"mixer.mu.{c}") for c in _MIXES])
+        if spec.mlp is not None and spec.mlp["kind"] == "moe":
+            for p in ("up", "down"):
+                mine[f"mlp.experts_{p}"] = torch.stack([mine.pop(f"mlp.experts.{e}.{p}")
+                                                        for e in range(spec.mlp["router"]["experts"])])
+        out.update({dst + k: v for k, v in mine.items()})
+    out.update({k: v for k, v in sd.items() if not k.startswith("model.layers.")})
     return out
+
+
+def _export_pafodra(sd, arch):
+    from .modeling import weight_owner
+    from ...ckpt.hf_import import PAFODRA_NAMES
+    back = {v: k for k, v in PAFODRA_NAMES.items()}
+    out = {"embed": sd["model.embed_tokens.weight"], "head": sd["lm_head.weight"]}
+    for n, suffix in (("weight", ""), ("bias", ".b"), ("alpha", ".alpha")):
+        out["final.norm" + suffix] = sd["model.norm." + n]
+    for i in range(len(arch.layers)):
+        if weight_owner(arch.layers, i) != i:
+            continue
+        pre = f"model.layers.{i}."
+        for k, v in sd.items():
+            if not k.startswith(pre):
+                continue
+            name = k[len(pre):]
+            if name == "mixer.mu":
+                out.update({f"l{i}.mix.mu.{c}": v[j] for j, c in enumerate(_MIXES)})
+            elif name in ("mlp.experts_up", "mlp.experts_down"):
+                out.update({f"l{i}.mlp.e{e}.{name[12:]}": w for e, w in enumerate(v)})
+            else:
+                out[f"l{i}.{back[name]}"] = v
+    return {k: v.contiguous() for k, v in out.items()}
 
 
 def export_state(sd, arch):
@@ -36,6 +91,8 @@ def export_state(sd, arch):
     fam = arch.family
     if fam in ("llama", "internlm"):
         return sd
+    if fam == "pafodra":
+        return _export_pafodra(sd, arch)
     out = {}
     L = arch.num_hidden_layers
     hq, hk, d, h = arch.num_attention_heads, arch.kv_heads, arch.head_dim, arch.hidden_size
@@ -87,6 +144,13 @@ def export_state(sd, arch):
 
 def export_config(arch):
     a = arch
+    if a.family == "pafodra":
+        layers = []
+        for l in a.layers:
+            e = {"type": l.type, "mixer": {k: v for k, v in l.mixer.items() if not k.endswith("_rank")}, "mlp": l.mlp}
+            layers.append(e if l.weights_of is None else dict(e, weights_of=l.weights_of))
+        return {"architecture": "Pafodra", "vocab": a.vocab_size, "width": a.hidden_size, "layers": layers,
+                "norm": {"eps": a.norm_eps}, "embedding": {"scale": a.embedding_scale}}
     if a.family == "qwen":
         return {"model_type": "qwen", "vocab_size": a.vocab_size, "hidden_size": a.hidden_size,
                 "intermediate_size": 2 * a.intermediate_size, "num_hidden_layers": a.num_hidden_layers,

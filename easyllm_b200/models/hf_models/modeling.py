@@ -17,16 +17,30 @@ from __future__ import annotations
 import json
 import math
 import os
-from dataclasses import dataclass
-from typing import Optional
+from dataclasses import dataclass, field
+from typing import List, Optional
 
 import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
 from ... import ops
+from ...ops import infer as iops
 from ...ops import reference as ref
 from ..layers import RotaryTables, alibi_slopes
+from .feedforward import DenseGLU, SparseMoE
+from .mixers import ChannelDelta, DynamicTanh, TimeMix
+from .state import DecodeState, KVRows
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a decoder whose layers differ: the mixer and its sizes, the feed-forward (None: no feed-forward),
+    and ``weights_of``, the layer whose tensors it uses (with a cache or state of its own)."""
+    type: str = "attention"               # attention | wkv | channel_delta
+    mixer: dict = field(default_factory=dict)
+    mlp: Optional[dict] = None
+    weights_of: Optional[int] = None
 
 
 @dataclass
@@ -54,6 +68,11 @@ class HFArch:
     pad_token_id: Optional[int] = None
     bos_token_id: Optional[int] = 1
     eos_token_id: Optional[int] = 2
+    # decoders whose layers differ: one spec per layer (None: num_hidden_layers equal attention + SwiGLU layers), run as
+    # parallel blocks x + mixer(norm x) + ff(norm x) on an fp32 stream
+    layers: Optional[List[LayerSpec]] = None
+    norm_eps: float = 1e-5                # eps of the mixers' own head norms
+    embedding_scale: float = 1.0
 
     @property
     def kv_heads(self):
@@ -66,7 +85,9 @@ class HFArch:
 
 def arch_from_hf_config(cfg: dict, family: Optional[str] = None) -> HFArch:
     """Translate a family's ``config.json`` into an HFArch."""
-    mt = (family or cfg.get("model_type") or "llama").lower()
+    mt = (family or cfg.get("model_type") or cfg.get("architecture") or "llama").lower()
+    if mt == "pafodra":
+        return _pafodra_arch(cfg)
     a = HFArch(family=mt)
     g = cfg.get
     if mt == "qwen":
@@ -107,6 +128,48 @@ def arch_from_hf_config(cfg: dict, family: Optional[str] = None) -> HFArch:
     return a
 
 
+_MIXER_SIZES = {"attention": ("heads", "kv_heads", "dim", "vdim", "scale"), "wkv": ("heads", "dim"),
+                "channel_delta": ("heads", "kv_heads", "dim", "vdim", "conv")}
+
+
+def _pafodra_arch(cfg: dict) -> HFArch:
+    """``config.json`` of a Pafodra model: vocab, width, norm.eps, embedding.scale and one entry per layer."""
+    layers = []
+    for i, e in enumerate(cfg["layers"]):
+        if e["type"] not in _MIXER_SIZES:
+            raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        missing = [k for k in _MIXER_SIZES[e["type"]] if k not in e["mixer"]]
+        if missing:
+            raise ValueError(f"layer {i} ({e['type']}): the config has no {missing}")
+        kv = e["mixer"].get("kv_heads")
+        if kv and e["mixer"]["heads"] % kv:
+            raise ValueError(f"layer {i}: {e['mixer']['heads']} heads do not divide into {kv} key/value heads")
+        mlp = e.get("mlp")
+        if mlp is not None and mlp["kind"] not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        w = e.get("weights_of")
+        if w is not None and not 0 <= w < len(cfg["layers"]):
+            raise ValueError(f"layer {i}: weights_of {w} is not a layer")
+        layers.append(LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else dict(mlp), w))
+    att = next((l.mixer for l in layers if l.type == "attention"), {})
+    return HFArch(family="pafodra", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layers=layers,
+                  num_hidden_layers=len(layers), num_attention_heads=att.get("heads", 1),
+                  num_key_value_heads=att.get("kv_heads", 1), norm_eps=cfg["norm"]["eps"],
+                  embedding_scale=cfg["embedding"]["scale"], position="none", bos_token_id=cfg.get("bos_token_id"),
+                  eos_token_id=cfg.get("eos_token_id"), pad_token_id=cfg.get("pad_token_id"))
+
+
+def weight_owner(layers, i):
+    """The layer whose tensors layer ``i`` uses (``weights_of`` followed to its end)."""
+    seen = set()
+    while layers[i].weights_of is not None and layers[i].weights_of != i:
+        if i in seen:
+            raise ValueError("weights_of runs in a circle")
+        seen.add(i)
+        i = layers[i].weights_of
+    return i
+
+
 class RMSNorm(nn.Module):
     def __init__(self, dim, eps, dtype):
         super().__init__()
@@ -120,21 +183,75 @@ class RMSNorm(nn.Module):
 
 
 class Attention(nn.Module):
-    def __init__(self, a: HFArch, dtype):
+    """Causal attention: GQA, RoPE / ALiBi / no positions, value heads of another size than the keys', a given score
+    scale, and a learned sink per head in the softmax denominator.  ``m``: sizes of this layer (None: the arch's)."""
+
+    def __init__(self, a: HFArch, dtype, m: Optional[dict] = None):
         super().__init__()
         self.a = a
-        d, hq, hk = a.head_dim, a.num_attention_heads, a.kv_heads
+        m = m or {"heads": a.num_attention_heads, "kv_heads": a.kv_heads, "dim": a.head_dim, "vdim": a.head_dim}
+        d, dv, hq, hk = m["dim"], m["vdim"], m["heads"], m["kv_heads"]
+        self.d, self.dv, self.hq, self.hk = d, dv, hq, hk
+        self.scale = float(m.get("scale", 1.0 / math.sqrt(d)))
         self.q_proj = nn.Linear(a.hidden_size, hq * d, bias=a.qkv_bias, dtype=dtype)
         self.k_proj = nn.Linear(a.hidden_size, hk * d, bias=a.qkv_bias, dtype=dtype)
-        self.v_proj = nn.Linear(a.hidden_size, hk * d, bias=a.qkv_bias, dtype=dtype)
-        self.o_proj = nn.Linear(hq * d, a.hidden_size, bias=a.o_bias, dtype=dtype)
+        self.v_proj = nn.Linear(a.hidden_size, hk * dv, bias=a.qkv_bias, dtype=dtype)
+        self.o_proj = nn.Linear(hq * dv, a.hidden_size, bias=a.o_bias, dtype=dtype)
+        self.sink = nn.Parameter(torch.zeros(hq)) if m.get("sink") else None
         self.rotary = RotaryTables(d, a.rope_theta, a.rope_scaling_factor, a.rope_dynamic_ntk_max_pos) \
             if a.position == "rope" else None
         self.slopes = torch.tensor(alibi_slopes(hq), dtype=torch.float32) if a.position == "alibi" else None
 
-    def forward(self, x, meta, cache=None):
+    def fused_groups(self):
+        ps = (self.q_proj, self.k_proj, self.v_proj)
+        return [[p.weight for p in ps]] + ([[p.bias for p in ps]] if self.a.qkv_bias else [])
+
+    def new_state(self, slots, capacity, device, dtype):
+        if self.a.use_cache_quantization:
+            from .kv_quant import QuantizedKV
+            return {"kq": QuantizedKV(slots, capacity, self.hk, self.d, device, dtype),
+                    "vq": QuantizedKV(slots, capacity, self.hk, self.dv, device, dtype), "len": 0}
+        return KVRows(slots, capacity, self.hk, self.d, self.dv, device, dtype)
+
+    def _split(self, qkv):
+        T, nq, nk = qkv.shape[0], self.hq * self.d, self.hk * self.d
+        return (qkv[:, :nq].view(T, self.hq, self.d), qkv[:, nq:nq + nk].view(T, self.hk, self.d),
+                qkv[:, nq + nk:].view(T, self.hk, self.dv))
+
+    def _attend(self, q, k, v, meta, cache):
+        """Serving attention: prompts that start here on the prefill kernel, everything else over the cached rows.
+        ``cache``: the layer's ``KVRows``, or None for packed sequences that keep nothing."""
+        T = q.shape[0]
+        sl = self.slopes.to(q.device) if self.slopes is not None else None
+        sink = self.sink.detach() if self.sink is not None else None
+        if cache is not None:
+            iops.kv_append(cache.k, cache.v, k, v, meta)
+        fresh = cache is None or (meta["fresh"] and not meta["one_token"])
+        if fresh and iops.prefill_kernel_ok(q, v):
+            row_start = meta["row_start"]
+            if row_start is None:
+                row_start = ops.cuda.row_start_of(meta["cu_seqlens"], T, q.device)
+            o = iops.attention_prefill(q, k, v, row_start, self.scale, sink, sl)
+        elif cache is not None:
+            o = iops.attention_rows(q, cache.k.view(-1, self.hk, self.d), cache.v.view(-1, self.hk, self.dv),
+                                    meta["kv_base"], meta["kv_len"], meta.get("kv_bound", meta["max_position"]),
+                                    self.scale, sink, sl)
+        else:
+            cu = meta["cu_seqlens"].long()
+            start = torch.repeat_interleave(cu[:-1], cu[1:] - cu[:-1], output_size=T)
+            n = torch.arange(T, device=q.device) - start + 1
+            o = iops.attention_rows(q, k, v, start.int(), n.int(), meta["max_seqlen"], self.scale, sink, sl)
+        return o.reshape(T, self.hq * self.dv)
+
+    def forward(self, x, meta, cache=None, residual=None):
+        """``residual``: fp32 stream the output projection is accumulated into (parallel blocks, inference only)."""
+        if residual is not None:
+            qkv = iops.linear_cat(x, [self.q_proj.weight, self.k_proj.weight, self.v_proj.weight],
+                                  [self.q_proj.bias, self.k_proj.bias, self.v_proj.bias] if self.a.qkv_bias else None)
+            o = self._attend(*self._split(qkv), meta, cache)
+            return iops.linear_add_(residual, o, self.o_proj.weight)
         a = self.a
-        d, hq, hk = a.head_dim, a.num_attention_heads, a.kv_heads
+        d, hq, hk = self.d, self.hq, self.hk
         T = x.shape[0]
         qkv = ops.linear_parts(x, (self.q_proj.weight, self.k_proj.weight, self.v_proj.weight),
                                (self.q_proj.bias, self.k_proj.bias, self.v_proj.bias) if a.qkv_bias else None)
@@ -151,13 +268,13 @@ class Attention(nn.Module):
             return ops.linear(o, self.o_proj.weight, self.o_proj.bias)
         if rope is not None:
             qkv = ops.rope_packed(qkv, cos, sin, pos, hq, hk, d)
-        q = qkv[:, :hq * d].view(T, hq, d)
-        k = qkv[:, hq * d:(hq + hk) * d].view(T, hk, d)
-        v = qkv[:, (hq + hk) * d:].view(T, hk, d)
+        q, k, v = self._split(qkv)
         if a.use_logn_attn and not self.training:
             logn = torch.clamp(torch.log(pos.float() + 1) / math.log(a.seq_length), min=1.0)
             q = (q.float() * logn.view(T, 1, 1)).to(q.dtype)
-        if cache is not None:
+        if isinstance(cache, KVRows):
+            o = self._attend(q, k, v, meta, cache)
+        elif cache is not None:               # dense batch of equal length in a dict: 8-bit cache, draft trees, prefixes
             B = meta["batch"]
             S = T // B
             p0 = cache["len"]
@@ -230,6 +347,9 @@ class DecoderLayer(nn.Module):
         self.input_layernorm = RMSNorm(a.hidden_size, a.rms_norm_eps, dtype)
         self.post_attention_layernorm = RMSNorm(a.hidden_size, a.rms_norm_eps, dtype)
 
+    def new_state(self, *a):
+        return self.self_attn.new_state(*a)
+
     def forward(self, delta, residual, meta, cache=None):
         if residual is None:
             h = delta
@@ -240,12 +360,52 @@ class DecoderLayer(nn.Module):
         return self.mlp(n2), h
 
 
+class ParallelLayer(nn.Module):
+    """``x + mixer(h) + ff(h)`` with one norm ``h = norm(x)``: both sublayers accumulate into the fp32 stream ``x``."""
+
+    def __init__(self, a: HFArch, spec: LayerSpec, dtype):
+        super().__init__()
+        m = spec.mixer
+        self.input_layernorm = DynamicTanh(a.hidden_size, dtype)
+        if spec.type == "attention":
+            self.mixer = Attention(a, dtype, dict(m, sink=True))
+        else:
+            self.mixer = {"wkv": TimeMix, "channel_delta": ChannelDelta}[spec.type](a.hidden_size, m, a.norm_eps, dtype)
+        self.mlp = None
+        if spec.mlp is not None:
+            self.mlp = DenseGLU(a.hidden_size, spec.mlp["ff"], "gelu_tanh", dtype) if spec.mlp["kind"] == "dense" \
+                else SparseMoE(a.hidden_size, spec.mlp, dtype)
+
+    def new_state(self, *a):
+        return self.mixer.new_state(*a)
+
+    def forward(self, x, _residual, meta, cache=None):
+        h = self.input_layernorm(x, self.mlp.out_bias if self.mlp is not None else None)
+        self.mixer(h, meta, cache, x)
+        if self.mlp is not None:
+            self.mlp(h, x)
+        return x, None
+
+
 class Decoder(nn.Module):
     def __init__(self, a: HFArch, dtype):
         super().__init__()
         self.embed_tokens = nn.Embedding(a.vocab_size, a.hidden_size, dtype=dtype)
-        self.layers = nn.ModuleList(DecoderLayer(a, dtype) for _ in range(a.num_hidden_layers))
-        self.norm = RMSNorm(a.hidden_size, a.rms_norm_eps, dtype)
+        self.embedding_scale, self.hybrid = a.embedding_scale, a.layers is not None
+        if self.hybrid:
+            own = {i: ParallelLayer(a, a.layers[i], dtype) for i in {weight_owner(a.layers, i) for i in range(len(a.layers))}}
+            # a layer with the weights of another one is the same module at two places, with a state at each
+            self.layers = nn.ModuleList(own[weight_owner(a.layers, i)] for i in range(len(a.layers)))
+            self.norm = DynamicTanh(a.hidden_size, dtype)
+        else:
+            self.layers = nn.ModuleList(DecoderLayer(a, dtype) for _ in range(a.num_hidden_layers))
+            self.norm = RMSNorm(a.hidden_size, a.rms_norm_eps, dtype)
+
+    def embed(self, ids):
+        """The residual stream the layers start from."""
+        if self.hybrid:
+            return iops.embed_scaled(ids.reshape(-1), self.embed_tokens.weight, self.embedding_scale)
+        return self.embed_tokens(ids.reshape(-1))
 
 
 def build_meta(input_ids, attention_mask=None, position_ids=None, cu_seqlens=None, device=None):
@@ -284,6 +444,14 @@ def build_meta(input_ids, attention_mask=None, position_ids=None, cu_seqlens=Non
     return meta
 
 
+def _penalise(logits, toks, seen, values):
+    """``logits[r, toks[r, c]] = values[r, c]`` where ``seen`` (padding columns must not touch their id's logit)."""
+    r, c = torch.nonzero(seen, as_tuple=True)
+    logits = logits.clone()
+    logits[r, toks[r, c]] = values[r, c]
+    return logits
+
+
 class CausalLM(nn.Module):
     def __init__(self, arch: HFArch, dtype=torch.float32):
         super().__init__()
@@ -315,8 +483,11 @@ class CausalLM(nn.Module):
         return F.normalize(w.float(), dim=-1).to(w.dtype) if self.arch.norm_head else w
 
     def hidden_states(self, input_ids, meta, caches=None, inputs_embeds=None):
-        x = inputs_embeds if inputs_embeds is not None else self.model.embed_tokens(input_ids.reshape(-1))
+        x = inputs_embeds if inputs_embeds is not None else self.model.embed(input_ids)
         x = x.reshape(-1, x.shape[-1])
+        if self.model.hybrid:
+            iops.no_grad_check(x, self.lm_head.weight)
+            x = x.float() if inputs_embeds is None else x.to(torch.float32, copy=True)     # the layers write into it
         delta, residual = x, None
         for i, layer in enumerate(self.model.layers):
             cache = caches[i] if caches is not None else None
@@ -331,6 +502,8 @@ class CausalLM(nn.Module):
 
     def forward(self, input_ids=None, attention_mask=None, labels=None, position_ids=None, cu_seqlens=None,
                 inputs_embeds=None, return_dict=True, **_):
+        if self.model.hybrid and labels is not None:
+            raise NotImplementedError(f"{self.arch.family}: the hybrid decoder layers are inference-only (no loss)")
         b, s = input_ids.shape
         dev = self.lm_head.weight.device
         # a batch handed over on the host is parsed there and copied (no read-back from the GPU per micro-batch)
@@ -338,6 +511,10 @@ class CausalLM(nn.Module):
         input_ids = input_ids.to(dev, non_blocking=True)
         if labels is not None:
             labels = labels.to(dev, non_blocking=True)
+        if self.model.hybrid:
+            with torch.no_grad():
+                h = self.hidden_states(input_ids, meta, inputs_embeds=inputs_embeds)
+                return {"logits": self.logits(h).view(b, s, -1)}
         h = self.hidden_states(input_ids, meta, inputs_embeds=inputs_embeds)
         out = {}
         if labels is not None:
@@ -355,12 +532,47 @@ class CausalLM(nn.Module):
         return out
 
     # ---- generation -----------------------------------------------------------------------------
+    def fuse_weights(self):
+        """Put the projections that are applied together next to each other in memory (once; a no-op afterwards)."""
+        for m in self.modules():
+            for group in getattr(m, "fused_groups", list)():
+                iops.make_adjacent_(group)
+
+    def new_state(self, slots, capacity):
+        """The cache / state manager of up to ``slots`` sequences of ``capacity`` tokens (it grows when that is not
+        enough)."""
+        self.fuse_weights()
+        return DecodeState(self, slots, capacity)
+
+    @torch.no_grad()
+    def step(self, state, slots, tokens, inputs_embeds=None):
+        """Run the next tokens of the sequences in ``slots`` as one batch, from what ``state`` holds of them.
+        ``tokens``: list of 1-D id tensors / lists (unequal lengths are packed, not padded), or one id per sequence as
+        a device tensor ``[n]``.  Returns the normed hidden rows of all tokens and the step's meta (``last_rows``: the
+        row of every sequence's last token)."""
+        dev = self.lm_head.weight.device
+        if torch.is_tensor(tokens):
+            counts, ids = [1] * len(slots), tokens.reshape(-1).to(dev)
+        else:
+            parts = [torch.as_tensor(t, dtype=torch.long).reshape(-1) for t in tokens]
+            counts, ids = [p.numel() for p in parts], torch.cat(parts).to(dev, non_blocking=True)
+        meta = state.step_meta(slots, counts)
+        return self.hidden_states(ids, meta, state.layers, inputs_embeds=inputs_embeds), meta
+
+    def logits(self, h):
+        """fp32 logits of hidden rows."""
+        if self.model.hybrid:
+            return iops.linear_f32(h, self.lm_head.weight)
+        return ops.linear(h, self.head_weight()).float()
+
     @torch.no_grad()
     def _decode_steps(self, input_ids, max_new_tokens=64, do_sample=False, temperature=1.0, top_k=0, top_p=0.0,
-                      eos_token_id=None, repetition_penalty=1.0, stop_words_ids=None, soft_prefix=None, **_):
-        """Greedy / sampled decoding with per-layer KV caches; yields the running ``[b, s]`` token tensor after
-        every new token.  A row ends at ``eos_token_id`` or when its tail equals one of ``stop_words_ids`` (token
-        sequences; the stop sequence stays in the output, later positions are filled with eos).
+                      eos_token_id=None, repetition_penalty=1.0, stop_words_ids=None, soft_prefix=None,
+                      attention_mask=None, **_):
+        """Greedy / sampled decoding from the cache / state manager; yields the running ``[b, s]`` token tensor after
+        every new token.  ``attention_mask``: rows of unequal length (padding on either side of ``input_ids``; new
+        tokens are appended after column ``s``).  A row ends at ``eos_token_id`` or when its tail equals one of
+        ``stop_words_ids`` (token sequences; the stop sequence stays in the output, later positions are filled with eos).
         ``soft_prefix``: ``{"embeds": [P, hidden]}`` (prompt tuning: virtual input embeddings in front of the
         prompt) or ``{"kv": [layers, 2, P, kv_heads, head_dim]}`` (prefix tuning: pre-filled cache entries)."""
         from ...infer.generation import sample_next
@@ -369,50 +581,53 @@ class CausalLM(nn.Module):
         stops = [torch.tensor(w, dtype=torch.long, device=input_ids.device) for w in (stop_words_ids or []) if len(w)]
         b, s = input_ids.shape
         dev, dt = input_ids.device, self.lm_head.weight.dtype
+        real = torch.ones(b, s, dtype=torch.bool) if attention_mask is None else attention_mask.bool().cpu()
+        prompts = [input_ids[i][real[i].to(dev)] for i in range(b)]
         soft = soft_prefix or {}
         pre_kv = soft.get("kv")
         pre_emb = soft.get("embeds")
         n_kv = 0 if pre_kv is None else pre_kv.shape[2]
         n_emb = 0 if pre_emb is None else pre_emb.shape[0]
-        room = s + max_new_tokens + n_kv + n_emb
-        if a.use_cache_quantization:
-            from .kv_quant import QuantizedKV
-            caches = [{"kq": QuantizedKV(b, room, a.kv_heads, a.head_dim, dev, dt),
-                       "vq": QuantizedKV(b, room, a.kv_heads, a.head_dim, dev, dt), "len": 0}
-                      for _ in range(a.num_hidden_layers)]
-        else:
-            caches = [{"k": torch.zeros(b, room, a.kv_heads, a.head_dim, dtype=dt, device=dev),
-                       "v": torch.zeros(b, room, a.kv_heads, a.head_dim, dtype=dt, device=dev), "len": 0}
-                      for _ in range(a.num_hidden_layers)]
+        state = self.new_state(b, s + max_new_tokens + n_kv + n_emb)
+        slots = [state.open() for _ in range(b)]
         if n_kv:
-            for l, c in enumerate(caches):
-                k0, v0 = (pre_kv[l, i].to(dt).unsqueeze(0).expand(b, -1, -1, -1) for i in (0, 1))
-                if "kq" in c:
-                    c["kq"].append(0, k0); c["vq"].append(0, v0)
+            for l, c in enumerate(state.layers):
+                k0, v0 = (pre_kv[l, i].to(dt) for i in (0, 1))
+                if isinstance(c, dict):
+                    c["kq"].append(0, k0.unsqueeze(0).expand(b, -1, -1, -1))
+                    c["vq"].append(0, v0.unsqueeze(0).expand(b, -1, -1, -1))
+                    c["len"] = n_kv
                 else:
-                    c["k"][:, :n_kv], c["v"][:, :n_kv] = k0, v0
-                c["len"] = n_kv
+                    c.load_prefix(slots, k0, v0)
+            for i in slots:
+                state.lengths[i] = n_kv
+        if a.use_cache_quantization and (not bool(real.all()) or slots != list(range(b))):
+            raise ValueError("the 8-bit cache holds a dense batch: prompts of one length only")
+        embeds = None
+        if n_emb:
+            embeds = torch.cat([torch.cat((pre_emb.to(dt), self.model.embed_tokens(p))) for p in prompts])
+            prompts = [torch.cat((p.new_zeros(n_emb), p)) for p in prompts]      # shapes only: the embeddings are given
         toks = input_ids
+        seen_mask = real.to(dev)
         done = torch.zeros(b, dtype=torch.bool, device=dev)
         fill = eos if eos is not None else 0
         for step in range(max_new_tokens):
-            inp = toks if step == 0 else toks[:, -1:]
-            p0 = n_kv if step == 0 else n_kv + n_emb + toks.shape[1] - 1
-            embeds = None
-            if step == 0 and n_emb:
-                embeds = torch.cat((pre_emb.to(dt).unsqueeze(0).expand(b, -1, -1), self.model.embed_tokens(inp)), 1)
-                inp = torch.cat((inp.new_zeros(b, n_emb), inp), 1)          # shapes only: the embeddings are given
-            pos = torch.arange(inp.shape[1], device=dev).unsqueeze(0).expand(b, -1) + p0
-            meta = build_meta(inp, None, pos)
-            h = self.hidden_states(inp, meta, caches, inputs_embeds=embeds)
-            logits = ops.linear(h.view(b, inp.shape[1], -1)[:, -1], self.head_weight()).float()
+            if step == 0:
+                h, meta = self.step(state, slots, prompts, inputs_embeds=embeds)
+                h = h[meta["last_rows"].to(h.device)]
+            else:
+                h, meta = self.step(state, slots, toks[:, -1])
+            logits = self.logits(h)
             if repetition_penalty != 1.0:
                 seen = torch.gather(logits, 1, toks)
-                logits.scatter_(1, toks, torch.where(seen > 0, seen / repetition_penalty, seen * repetition_penalty))
+                pen = torch.where(seen > 0, seen / repetition_penalty, seen * repetition_penalty)
+                logits = logits.scatter(1, toks, torch.where(seen_mask, pen, seen)) if bool(real.all()) else \
+                    _penalise(logits, toks, seen_mask, pen)
             nxt = sample_next(logits, temperature, top_k, top_p, greedy=not do_sample)
             if eos is not None or stops:
                 nxt = torch.where(done, torch.full_like(nxt, fill), nxt)
             toks = torch.cat((toks, nxt.unsqueeze(1)), 1)
+            seen_mask = F.pad(seen_mask, (0, 1), value=True)
             if eos is not None:
                 done |= nxt == eos
             new_len = toks.shape[1] - s
@@ -425,7 +640,7 @@ class CausalLM(nn.Module):
 
     def generate(self, input_ids, attention_mask=None, max_new_tokens=64, num_beams=1, **kw):
         toks = input_ids
-        for toks in self._decode_steps(input_ids, max_new_tokens=max_new_tokens, **kw):
+        for toks in self._decode_steps(input_ids, max_new_tokens=max_new_tokens, attention_mask=attention_mask, **kw):
             pass
         return toks
 
@@ -450,18 +665,20 @@ class CausalLM(nn.Module):
 
     @classmethod
     def from_pretrained(cls, path, family=None, torch_dtype=torch.float32, arch_overrides=None, **_):
-        from .io import import_state
+        from .io import import_state, sizes_from_state
+        from ...ckpt.hf_import import load_hf_state
         with open(os.path.join(path, "config.json")) as f:
             cfg = json.load(f)
         arch = arch_from_hf_config(cfg, family)
+        raw = load_hf_state(path)
+        sizes_from_state(arch, raw)
         for k, v in (arch_overrides or {}).items():
             setattr(arch, k, v)
         if isinstance(torch_dtype, str):
             torch_dtype = getattr(torch, torch_dtype.replace("torch.", ""))
         model = cls(arch, torch_dtype)
-        from ...ckpt.hf_import import load_hf_state
-        sd = import_state(load_hf_state(path), arch)
-        missing, unexpected = model.load_state_dict({k: v.to(torch_dtype) for k, v in sd.items()}, strict=False)
+        sd = import_state(raw, arch)
+        missing, unexpected = model.load_state_dict(sd, strict=False)      # copies into each parameter's own dtype
         missing = [m for m in missing if not (arch.tie_word_embeddings and m == "lm_head.weight")]
         if missing or unexpected:
             raise RuntimeError(f"from_pretrained({path}): missing {missing[:8]}, unexpected {unexpected[:8]}")

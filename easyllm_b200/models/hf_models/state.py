@@ -1,0 +1,133 @@
+"""What running sequences keep between steps: slots, per-layer caches and states, and the index of one step.
+
+``DecodeState`` is the manager.  A sequence opens a slot, every step appends tokens to some slots, and closing the slot
+gives it back; a slot that is used again starts from position 0, which every layer takes as "nothing before".  Each
+layer contributes one state object through ``layer.new_state``:
+
+* ``KVRows``: keys and values, ``[slots, capacity, kv_heads, dim]``, grown in whole blocks of positions;
+* ``SlotTensors``: fixed-size tensors per slot (recurrent matrices, last inputs of a short convolution or a token shift);
+* a plain dict (the 8-bit cache of Qwen): dense batches of equal length only.
+
+``DecodeState.step_meta`` is the packed description of one step that the layers read.  All index tensors are built on
+the host and copied once; a decode step (one token a sequence) of the same slots can be advanced in place on the
+device (``advance``), so its kernels can be replayed from a CUDA graph.
+"""
+from __future__ import annotations
+
+import torch
+
+BLOCK = 256          # positions a key/value cache grows by
+
+
+class KVRows:
+    def __init__(self, slots, capacity, kv_heads, dim, vdim, device, dtype):
+        self.k = torch.zeros(slots, capacity, kv_heads, dim, dtype=dtype, device=device)
+        self.v = torch.zeros(slots, capacity, kv_heads, vdim, dtype=dtype, device=device)
+
+    def grow(self, slots, capacity):
+        for name in ("k", "v"):
+            old = getattr(self, name)
+            new = old.new_zeros(slots, capacity, *old.shape[2:])
+            new[:old.shape[0], :old.shape[1]] = old
+            setattr(self, name, new)
+
+    def load_prefix(self, slots, k, v):
+        """Fill positions ``0 .. n`` of ``slots`` with given keys / values ``[n, kv_heads, dim]`` (prefix tuning)."""
+        for s in slots:
+            self.k[s, :k.shape[0]], self.v[s, :v.shape[0]] = k.to(self.k.dtype), v.to(self.v.dtype)
+
+
+class SlotTensors:
+    def __init__(self, slots, device, **shapes):
+        """``name=(shape, dtype)`` per tensor; each becomes an attribute ``[slots, *shape]``."""
+        self.names = list(shapes)
+        for name, (shape, dtype) in shapes.items():
+            setattr(self, name, torch.zeros(slots, *shape, dtype=dtype, device=device))
+
+    def grow(self, slots, capacity):
+        for name in self.names:
+            old = getattr(self, name)
+            new = old.new_zeros(slots, *old.shape[1:])
+            new[:old.shape[0]] = old
+            setattr(self, name, new)
+
+
+class DecodeState:
+    def __init__(self, model, slots, capacity, device=None, dtype=None):
+        w = model.lm_head.weight
+        self.device, self.dtype = device or w.device, dtype or w.dtype
+        self.capacity = -(-capacity // BLOCK) * BLOCK
+        self.layers = [layer.new_state(slots, self.capacity, self.device, self.dtype) for layer in model.model.layers]
+        self.lengths = [0] * slots
+        self.free = list(range(slots - 1, -1, -1))
+
+    @property
+    def slots(self):
+        return len(self.lengths)
+
+    def open(self):
+        """A slot for a new sequence (the manager grows when none is free)."""
+        if not self.free:
+            n = self.slots
+            self._grow(2 * n, self.capacity)
+            self.lengths += [0] * n
+            self.free = list(range(2 * n - 1, n - 1, -1))
+        s = self.free.pop()
+        self.lengths[s] = 0
+        return s
+
+    def close(self, slot):
+        self.lengths[slot] = 0
+        self.free.append(slot)
+
+    def reserve(self, length):
+        """Room for sequences of ``length`` tokens."""
+        if length > self.capacity:
+            self._grow(self.slots, -(-max(length, 2 * self.capacity) // BLOCK) * BLOCK)
+
+    def _grow(self, slots, capacity):
+        for st in self.layers:
+            if not hasattr(st, "grow"):
+                raise ValueError("this cache cannot grow: it holds one dense batch of a fixed size")
+            st.grow(slots, capacity)
+        self.capacity = capacity
+
+    # ---- one step ------------------------------------------------------------------------------
+    def step_meta(self, slots, counts):
+        """Packed meta of a step that appends ``counts[i]`` tokens to ``slots[i]``; the lengths advance."""
+        if len(set(slots)) != len(slots) or any(c < 1 for c in counts):
+            raise ValueError("a step brings at least one token to each of its (distinct) sequences")
+        start = [self.lengths[s] for s in slots]
+        self.reserve(max(p + c for p, c in zip(start, counts)))
+        dev, S, T = self.device, len(slots), sum(counts)
+        cu = [0]
+        for c in counts:
+            cu.append(cu[-1] + c)
+        n = torch.tensor(counts)
+        sl, p0 = torch.tensor(slots), torch.tensor(start)
+        first = torch.tensor(cu[:-1])
+        pos = torch.arange(T) - torch.repeat_interleave(first - p0, n, output_size=T)
+        # one host buffer, one copy: sequence borders, slots, start positions | positions, first row of the sequence,
+        # row of its first key, keys
+        tok_slot = torch.repeat_interleave(sl, n, output_size=T)
+        rows = torch.repeat_interleave(first, n, output_size=T)
+        buf = torch.cat((torch.tensor(cu), sl, p0, pos, rows, tok_slot * self.capacity, pos + 1)).to(torch.int32)
+        if dev.type == "cuda":
+            buf = buf.pin_memory().to(dev, non_blocking=True)
+        parts = buf.split([S + 1, S, S, T, T, T, T])
+        for s, c in zip(slots, counts):
+            self.lengths[s] += c
+        fresh = not any(start)
+        return {"cu_seqlens": parts[0], "seq_slot": parts[1], "seq_pos0": parts[2], "position_ids": parts[3],
+                "row_start": parts[4], "kv_base": parts[5], "kv_len": parts[6], "max_seqlen": max(counts),
+                "max_position": max(p + c for p, c in zip(start, counts)), "batch": S, "fresh": fresh,
+                "one_token": T == S, "kv_capacity": self.capacity,
+                "last_rows": torch.tensor(cu[1:]) - 1, "slots": list(slots)}
+
+    def advance(self, meta):
+        """Turn the meta of a one-token step into that of the next one, on the device."""
+        for s in meta["slots"]:
+            self.lengths[s] += 1
+        meta["seq_pos0"].add_(1)
+        meta["position_ids"].add_(1)
+        meta["kv_len"].add_(1)
