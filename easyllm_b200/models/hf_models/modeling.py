@@ -559,6 +559,7 @@ class CausalLM(nn.Module):
         meta = state.step_meta(slots, counts)
         return self.hidden_states(ids, meta, state.layers, inputs_embeds=inputs_embeds), meta
 
+    @torch.no_grad()
     def logits(self, h):
         """fp32 logits of hidden rows."""
         if self.model.hybrid:

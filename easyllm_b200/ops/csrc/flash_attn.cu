@@ -1,5 +1,6 @@
 // Causal flash attention forward on tcgen05 / TMEM for sm_100a: packed variable-length
-// documents, MHA and GQA, head_dim 128, bf16 in/out, fp32 softmax.
+// documents, MHA and GQA, key and value heads of up to 128 (multiples of 8, sizes of their own), bf16 in/out, fp32
+// softmax with an optional learned sink per head in the denominator.
 //
 // One CTA per (pair of adjacent 128-query tiles, query head); 320 threads:
 //   warp 0     TMA: both Q tiles once, then K tiles (128 keys) through a 2-stage ring and V tiles one at a time
@@ -18,6 +19,9 @@
 // visible to query i iff row_start[i] <= j <= i, so tiles may straddle document boundaries.
 // ALiBi: with per-head slopes the score of (query i, key j) gets the bias slope_h * (j - i) before the softmax
 // (llm/models/hf_models/baichuan2/model_13b/modeling_baichuan.py:63-73 builds the same bias as a mask tensor).
+//
+// Head sizes below 128: the tensor maps are [dim, heads, rows], so a 64-column box that reaches past a head's end is
+// zero-filled by the TMA unit; the score product runs ceil(dim / 16) k-steps and P·V is ceil(vdim / 16) * 16 wide.
 //
 // Replaces flash_attn_varlen_{qkv,kv}packed_func of the reference
 // (llm/models/mg_models/llama/transformer.py:65-143).
@@ -72,7 +76,8 @@ __global__ void __launch_bounds__(kFaThreads, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
                  float* __restrict__ lse, const int* __restrict__ row_start, int T, int Hq, int Hk,
-                 float scale_log2, const float* __restrict__ alibi_slopes, int* __restrict__ err) {
+                 int d, int dv, float scale_log2, const float* __restrict__ alibi_slopes,
+                 const float* __restrict__ sink, int* __restrict__ err) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* sQ = smem;                          // 2 query tiles
@@ -93,6 +98,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
   for (int t = 0; t < 2; ++t) n_kv[t] = fa_num_kv_tiles(q0 + t * kFaM, T, kv_lo);
   const int n_kv_max = max(n_kv[0], n_kv[1]);
+  const bool wide_k = d > 64, wide_v = dv > 64;   // heads of up to 64 use one 64-column half of a tile
+  const uint32_t k_bytes = wide_k ? kFaTileBytes : kFaTileBytes / 2, v_bytes = wide_v ? kFaTileBytes : kFaTileBytes / 2;
 
   if (threadIdx.x == 0) {
     mbar_init(&sh->q_full, 1);
@@ -125,20 +132,20 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   } else if (warp == 0) {
     if (lane == 0) {
       bool ok = true;
-      mbar_expect_tx(&sh->q_full, 2 * kFaTileBytes);
+      mbar_expect_tx(&sh->q_full, 2 * k_bytes);
 #pragma unroll
       for (int t = 0; t < 2; ++t) {            // rows past T are zero-filled by the TMA unit
-        tma_load_2d(sQ + t * kFaTileBytes, &tmQ, &sh->q_full, h * kFaD, q0 + t * kFaM);
-        tma_load_2d(sQ + t * kFaTileBytes + kFaTileBytes / 2, &tmQ, &sh->q_full, h * kFaD + 64, q0 + t * kFaM);
+        tma_load_3d(sQ + t * kFaTileBytes, &tmQ, &sh->q_full, 0, h, q0 + t * kFaM);
+        if (wide_k) tma_load_3d(sQ + t * kFaTileBytes + kFaTileBytes / 2, &tmQ, &sh->q_full, 64, h, q0 + t * kFaM);
       }
       // K runs one tile ahead of V: K(j+1) is requested as soon as S(j-1) released its stage, before the
       // loader blocks on the single V stage (free only once PV(j-1) is done)
       auto load_k = [&](int j) -> bool {
         const int s = j & 1;
         if (!mbar_wait(&sh->k_empty[s], ((j >> 1) & 1) ^ 1, abort_flag)) return false;
-        mbar_expect_tx(&sh->k_full[s], kFaTileBytes);
-        tma_load_2d(sK + s * kFaTileBytes, &tmK, &sh->k_full[s], kvh * kFaD, kv_lo + j * kFaN);
-        tma_load_2d(sK + s * kFaTileBytes + kFaTileBytes / 2, &tmK, &sh->k_full[s], kvh * kFaD + 64, kv_lo + j * kFaN);
+        mbar_expect_tx(&sh->k_full[s], k_bytes);
+        tma_load_3d(sK + s * kFaTileBytes, &tmK, &sh->k_full[s], 0, kvh, kv_lo + j * kFaN);
+        if (wide_k) tma_load_3d(sK + s * kFaTileBytes + kFaTileBytes / 2, &tmK, &sh->k_full[s], 64, kvh, kv_lo + j * kFaN);
         return true;
       };
       if (n_kv_max > 0) ok = load_k(0);
@@ -146,9 +153,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         const int k0 = kv_lo + j * kFaN;
         if (j + 1 < n_kv_max && !load_k(j + 1)) { ok = false; break; }
         if (!mbar_wait(&sh->v_empty, (j & 1) ^ 1, abort_flag)) { ok = false; break; }
-        mbar_expect_tx(&sh->v_full, kFaTileBytes);
-        tma_load_2d(sV, &tmV, &sh->v_full, kvh * kFaD, k0);
-        tma_load_2d(sV + kFaTileBytes / 2, &tmV, &sh->v_full, kvh * kFaD + 64, k0);
+        mbar_expect_tx(&sh->v_full, v_bytes);
+        tma_load_3d(sV, &tmV, &sh->v_full, 0, kvh, k0);
+        if (wide_v) tma_load_3d(sV + kFaTileBytes / 2, &tmV, &sh->v_full, 64, kvh, k0);
       }
       if (!ok) {
         sh->abort_flag = 1;
@@ -158,7 +165,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, 128, false, true);
+      const uint32_t idesc_o = make_idesc_bf16(128, (dv + 15) / 16 * 16, false, true);
+      const int k_steps = (d + 15) / 16;
       bool ok = mbar_wait(&sh->q_full, 0, abort_flag);
       const uint32_t v_addr = smem_u32(sV);
       // S_t(j) = Q_t K_j^T for both query tiles that still walk key tile j
@@ -175,6 +183,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           const uint32_t q_addr = smem_u32(sQ + t * kFaTileBytes);
 #pragma unroll
           for (int k = 0; k < 8; ++k) {
+            if (k >= k_steps) break;
             const uint32_t off = (k >> 2) * (kFaTileBytes / 2) + (k & 3) * 32;
             umma_bf16(tmem_base + t * 128, make_smem_desc(q_addr + off, 16, 1024),
                       make_smem_desc(k_addr + off, 16, 1024), idesc_s, k != 0);
@@ -293,7 +302,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       if (j > 0 && __any_sync(0xffffffffu, grow)) {
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c * 32 < dv; ++c) {
           uint32_t v[32];
           tmem_ld_32x32(t_o + c * 32, v);
           tmem_ld_wait();
@@ -325,16 +334,19 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       if (!mbar_wait(&sh->pv_done[t], (my_n - 1) & 1, abort_flag)) fail();
       tc_fence_after();
       if (ok && !*abort_flag) {
+        // the sink is one more term of the denominator, without a key or a value
+        if (sink != nullptr) l += exp2f(sink[h] * 1.4426950408889634f - m_used);
         const float inv_l = row_valid ? 1.f / l : 0.f;
-        __nv_bfloat16* orow = out + ((size_t)row * Hq + h) * kFaD;
+        __nv_bfloat16* orow = out + ((size_t)row * Hq + h) * dv;
 #pragma unroll 1
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c * 32 < dv; ++c) {
           uint32_t v[32];
           tmem_ld_32x32(t_o + c * 32, v);
           tmem_ld_wait();
           if (row_valid) {
 #pragma unroll
             for (int g = 0; g < 4; ++g) {
+              if (c * 32 + g * 8 >= dv) break;
               float f[8];
 #pragma unroll
               for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g * 8 + i]) * inv_l;
@@ -342,7 +354,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             }
           }
         }
-        if (row_valid) lse[(size_t)h * T + row] = m_used * 0.6931471805599453f + logf(l);
+        if (row_valid && lse != nullptr) lse[(size_t)h * T + row] = m_used * 0.6931471805599453f + logf(l);
       }
     }
   }
@@ -362,8 +374,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   }
 }
 
-int make_tmap_bf16_2d(CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint64_t row_stride_bytes,
-                      uint32_t box_inner, uint32_t box_outer);
+int make_tmap_bf16_heads(CUtensorMap* map, const void* ptr, uint64_t dim, uint64_t heads, uint64_t rows,
+                         uint64_t row_stride_bytes, uint32_t box_dim, uint32_t box_rows);
 
 }  // namespace ell
 
@@ -399,21 +411,21 @@ ELL_API int ell_flash_fwd_plan(const int* row_start, int T, int* out) {
   return n_pairs;
 }
 
-// q [T, Hq, 128] / k, v [T, Hk, 128] bf16 with row strides (in elements) q_stride / kv_stride (views
-// into the packed QKV GEMM output are fine); out [T, Hq, 128] contiguous; lse [Hq, T] fp32;
-// row_start [T] int32 (document start of every token).  Causal.
-// alibi_slopes: fp32 [Hq] or null.
+// q [T, Hq, d], k [T, Hk, d], v [T, Hk, dv] bf16 with row strides (in elements) q_stride / k_stride / v_stride (views
+// into the packed QKV GEMM output are fine), d and dv multiples of 8 up to 128; out [T, Hq, dv] contiguous; lse [Hq, T]
+// fp32 or null; row_start [T] int32 (document start of every token).  Causal.
+// alibi_slopes, sink: fp32 [Hq] or null.
 ELL_API int ell_flash_attn_fwd(const void* q, const void* k, const void* v, void* out, float* lse, const int* row_start,
-                               int T, int Hq, int Hk, int q_stride, int kv_stride, float scale,
-                               const float* alibi_slopes, int* err, cudaStream_t stream) {
+                               int T, int Hq, int Hk, int d, int dv, int q_stride, int k_stride, int v_stride, float scale,
+                               const float* alibi_slopes, const float* sink, int* err, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (Hq % Hk) return -2;
+  if (Hq % Hk || d < 8 || d > kFaD || d % 8 || dv < 8 || dv > kFaD || dv % 8) return -2;
   CUtensorMap tq, tk, tv;
-  int rc = make_tmap_bf16_2d(&tq, q, (uint64_t)Hq * kFaD, (uint64_t)T, (uint64_t)q_stride * 2, 64, 128);
+  int rc = make_tmap_bf16_heads(&tq, q, d, Hq, T, (uint64_t)q_stride * 2, 64, 128);
   if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tk, k, (uint64_t)Hk * kFaD, (uint64_t)T, (uint64_t)kv_stride * 2, 64, 128);
+  rc = make_tmap_bf16_heads(&tk, k, d, Hk, T, (uint64_t)k_stride * 2, 64, 128);
   if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tv, v, (uint64_t)Hk * kFaD, (uint64_t)T, (uint64_t)kv_stride * 2, 64, 128);
+  rc = make_tmap_bf16_heads(&tv, v, dv, Hk, T, (uint64_t)v_stride * 2, 64, 128);
   if (rc) return rc;
   static bool configured = false;
   if (!configured) {
@@ -423,6 +435,7 @@ ELL_API int ell_flash_attn_fwd(const void* q, const void* k, const void* v, void
   }
   dim3 grid((T + 2 * kFaM - 1) / (2 * kFaM), Hq);
   flash_fwd_kernel<<<grid, kFaThreads, kFaSmemBytes, stream>>>(tq, tk, tv, (__nv_bfloat16*)out, lse, row_start, T, Hq,
-                                                               Hk, scale * 1.4426950408889634f, alibi_slopes, err);
+                                                               Hk, d, dv, scale * 1.4426950408889634f, alibi_slopes,
+                                                               sink, err);
   return launch_status();
 }

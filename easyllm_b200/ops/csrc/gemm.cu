@@ -117,7 +117,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   GemmShared* sh = reinterpret_cast<GemmShared*>(sC + 2 * kEpiBufBytes);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int tiles_m = (M + kBM - 1) / kBM, tiles_n = (N + BN - 1) / BN;
+  const int tiles_m = FUSE == kFuseGroup ? min(*fuse.n_row_tiles, (M + kBM - 1) / kBM) : (M + kBM - 1) / kBM;
+  const int tiles_n = (N + BN - 1) / BN;
   const int num_tiles = tiles_m * tiles_n;
   const int num_kb = (K + kBK - 1) / kBK;
   const int n_comm = FUSE == kFuseNone ? 0 : fuse.n_comm;
@@ -171,6 +172,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         const uint32_t stage_bytes = kABytes + (uint32_t)u.bn * kBK * 2;
         const CUtensorMap* a_map = &tmA;
         int a_row = m0;
+        // a B tile may reach into the next expert's rows: those columns lie past N and are not stored
+        const int b_row = FUSE == kFuseGroup ? fuse.tile_expert[mt] * N + n0 : n0;
         if (FUSE == kFuseAG) {
           // rows of this tile come from rank `src`: the local shard is read in place, a remote shard
           // from the local gathered buffer once the peer's copy of this tile is flagged
@@ -205,7 +208,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               tma_load_2d(a_dst + i * (64 * kBK * 2), &tmA, &sh->full[stage], m0 + i * 64, kb * kBK);
           }
           if (!B_MN) {
-            tma_load_2d(b_dst, b_map, &sh->full[stage], kb * kBK, n0);
+            tma_load_2d(b_dst, b_map, &sh->full[stage], kb * kBK, b_row);
           } else {
 #pragma unroll
             for (int i = 0; i < BN / 64; ++i)
@@ -324,6 +327,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               const int col = n0 + j * 64 + c;
               const float b = col < N ? __bfloat162float(bias[col]) : 0.f;
               r[c] = __float_as_uint(__uint_as_float(r[c]) + b);
+            }
+          }
+          if (FUSE == kFuseGroup && fuse.row_scale != nullptr) {
+            const float sc = fuse.row_scale[m0 + row_in_tile];
+#pragma unroll
+            for (int c = 0; c < 64; ++c) {
+              const float x = sc * fmaxf(__uint_as_float(r[c]), 0.f);
+              r[c] = __float_as_uint(x * x);
             }
           }
           if (OUT == kOutBf16CE) {
@@ -516,6 +527,22 @@ static int make_tmap_2d(CUtensorMap* map, CUtensorMapDataType dt, const void* pt
   return r == CUDA_SUCCESS ? 0 : -12;
 }
 
+// 3-D bf16 tensor map over [rows, heads, dim] (dim contiguous, heads packed): boxes of one head, zero-filled past `dim`.
+int make_tmap_bf16_heads(CUtensorMap* map, const void* ptr, uint64_t dim, uint64_t heads, uint64_t rows,
+                         uint64_t row_stride_bytes, uint32_t box_dim, uint32_t box_rows) {
+  EncodeTiledFn fn = get_encode_fn();
+  if (!fn) return -10;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (row_stride_bytes & 15) || ((dim * 2) & 15)) return -11;
+  cuuint64_t dims[3] = {dim, heads, rows};
+  cuuint64_t strides[2] = {dim * 2, row_stride_bytes};
+  cuuint32_t box[3] = {box_dim, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -12;
+}
+
 template <int BN, bool A_MN, bool B_MN, int OUT, bool HAS_BIAS, int FUSE = kFuseNone>
 static int launch_gemm(const CUtensorMap& tA, const CUtensorMap& tB, const CUtensorMap& tC, const FuseArgs& fuse,
                        const __nv_bfloat16* bias, int M, int N, int K, int ldc, int* err, int max_ctas,
@@ -667,10 +694,35 @@ ELL_API int ell_gemm_bf16(const void* A, const void* B, void* C, const void* bia
   ELL_GEMM_CASE(BN_, true, true, kOutF32Accum, false) \
   ELL_GEMM_CASE(BN_, true, true, kOutF32, false)    \
   ELL_GEMM_CASE(BN_, false, false, kOutF32, false)  \
+  ELL_GEMM_CASE(BN_, false, false, kOutF32Accum, false) \
   ELL_GEMM_CASE(BN_, false, true, kOutF32, false)
   ELL_GEMM_BN(256)
   ELL_GEMM_BN(128)
   return -3;
+}
+
+// Grouped product for rows sorted by expert: C[rows, N] (bf16) = A[rows, K] · W[expert of the row tile][N, K]^T, where
+// every expert's rows start at a multiple of 128.  W is [experts * N, K]; `rows` is the capacity of A and C (a multiple
+// of 128), *n_row_tiles the 128-row tiles in use.  row_scale (fp32 [rows] or null): C = (row_scale relu(.))^2.
+ELL_API int ell_gemm_grouped(const void* A, const void* W, void* C, const int* tile_expert, const int* n_row_tiles,
+                             const float* row_scale, int rows, int N, int K, int experts, int* err, cudaStream_t stream) {
+  if (rows <= 0 || N <= 0 || K <= 0) return 0;
+  if (rows % kBM || N % 8 || K % 8) return -2;
+  const int BN = N > 128 ? 256 : 128;
+  CUtensorMap tA, tB, tC;
+  int rc = make_tmap_bf16_2d(&tA, A, (uint64_t)K, (uint64_t)rows, (uint64_t)K * 2, kBK, kBM);
+  if (rc) return rc;
+  rc = make_tmap_bf16_2d(&tB, W, (uint64_t)K, (uint64_t)experts * N, (uint64_t)K * 2, kBK, BN);
+  if (rc) return rc;
+  rc = make_tmap_bf16_2d(&tC, C, (uint64_t)N, (uint64_t)rows, (uint64_t)N * 2, 64, 128);
+  if (rc) return rc;
+  FuseArgs f{};
+  f.tile_expert = tile_expert;
+  f.n_row_tiles = n_row_tiles;
+  f.row_scale = row_scale;
+  if (BN == 256)
+    return launch_gemm<256, false, false, kOutBf16, false, kFuseGroup>(tA, tB, tC, f, nullptr, rows, N, K, N, err, sm_count(), stream);
+  return launch_gemm<128, false, false, kOutBf16, false, kFuseGroup>(tA, tB, tC, f, nullptr, rows, N, K, N, err, sm_count(), stream);
 }
 
 // Column tiles the cross-entropy epilogue produces partials for (BN = 256).

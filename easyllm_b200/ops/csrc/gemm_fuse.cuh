@@ -18,6 +18,9 @@
 //            above, after which each owner leaves the reduced tile in its staging buffer and raises a second
 //            flag on every peer; all ranks then pull the tiles they do not own (peer bulk loads) into their
 //            full-size output.  Two-shot: each byte crosses NVLink once per phase.
+//  kFuseGroup  no collective: a grouped product for rows sorted by expert.  Row tile i multiplies the weight rows of
+//            expert tile_expert[i] of a stacked [experts * N, K] operand; the number of row tiles is read on the device.
+//            With row_scale the epilogue writes (row_scale relu(c))^2.
 // Flags are epoch counters that only grow; a per-peer `done` word tells a producer that the consumer has
 // finished the previous epoch before a buffer is overwritten.  Every wait is bounded and reports through the
 // error word.  Tensor maps only ever cover this GPU's memory and no load names more than one destination CTA.
@@ -41,7 +44,7 @@ constexpr int kEpiBufBytes = 128 * 64 * 2; // one 128x64 bf16 store box
 // of the rounded logits, computed in the epilogue while the tile is in registers.
 enum GemmOut { kOutBf16 = 0, kOutF32Accum = 1, kOutF32 = 2, kOutBf16CE = 3 };
 enum GemmErr { kErrProducer = 1, kErrMma = 2, kErrEpilogue = 3, kErrComm = 4, kErrFlagWait = 5, kErrBounds = 6 };
-enum GemmFuse { kFuseNone = 0, kFuseAG = 1, kFuseRS = 2, kFuseAR = 3, kFuseAGK = 4 };
+enum GemmFuse { kFuseNone = 0, kFuseAG = 1, kFuseRS = 2, kFuseAR = 3, kFuseAGK = 4, kFuseGroup = 5 };
 constexpr int kMaxTp = 8;
 
 struct FuseArgs {
@@ -67,6 +70,9 @@ struct FuseArgs {
   int shard_k;                           // row length of x_local when this struct describes a bare push (see below)
   int k_passes;                          // AGK: 2 walks every tile twice (local half of the k-range first), 1 once
   unsigned long long data_bytes;         // size of each data_ptrs[] buffer: every computed offset is checked against it
+  const int* tile_expert;                // Group: expert of every row tile
+  const int* n_row_tiles;                // Group: number of row tiles in use
+  const float* row_scale;                // Group: per-row scale of the squared-relu epilogue, or null
   int rs_lag_q;                          // CTA-pair reduce-scatter: own tiles trail the peers' by this many quarter waves (0: default)
 };
 

@@ -1110,6 +1110,7 @@ ELL_API int ell_gemm_bf16_pair(const void* A, const void* B, void* C, const void
   ELL_PAIR_CASE(true, true, kOutF32Accum, false)
   ELL_PAIR_CASE(true, true, kOutF32, false)
   ELL_PAIR_CASE(false, false, kOutF32, false)
+  ELL_PAIR_CASE(false, false, kOutF32Accum, false)
   ELL_PAIR_CASE(false, true, kOutF32, false)
 #undef ELL_PAIR_CASE
   return -3;

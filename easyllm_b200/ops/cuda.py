@@ -16,6 +16,7 @@ import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _LIB_PATH = os.path.join(_HERE, "libeasyllm_b200.so")
+_SERVE_LIB_PATH = os.path.join(_HERE, "libeasyllm_b200_serve.so")      # the serving kernels alone (ops.build)
 _lib = None
 LAUNCHES = 0
 _err_flags = {}
@@ -27,17 +28,18 @@ class KernelError(RuntimeError):
 
 
 def available():
-    return os.path.exists(_LIB_PATH)
+    return os.path.exists(_LIB_PATH) or os.path.exists(_SERVE_LIB_PATH)
 
 
 def lib():
     global _lib
     if _lib is None:
-        if not os.path.exists(_LIB_PATH):
+        if not available():
             raise KernelError(f"{_LIB_PATH} is missing: run `python -m easyllm_b200.ops.build` "
                               "(or __graft_entry__.build()) before using the CUDA ops")
-        _lib = ctypes.CDLL(_LIB_PATH)
-        _lib.ell_rmsnorm_bwd_scratch_elems.restype = c_longlong
+        _lib = ctypes.CDLL(_LIB_PATH if os.path.exists(_LIB_PATH) else _SERVE_LIB_PATH)
+        for name in ("ell_rmsnorm_bwd_scratch_elems", "ell_attn_rows_scratch"):
+            getattr(_lib, name).restype = c_longlong
     return _lib
 
 
@@ -501,22 +503,25 @@ def _slopes(alibi_slopes, Hq, device):
     return sl
 
 
-def flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes=None):
-    """q [T,Hq,128], k/v [T,Hk,128] (last two dims contiguous, any row stride) → (out, lse [Hq,T]).
-    ``alibi_slopes`` fp32 [Hq]: adds ``slope_h · (key − query)`` to the scores."""
+def flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes=None, sink=None):
+    """q [T,Hq,D], k [T,Hk,D], v [T,Hk,Dv] (heads packed in a row, any row stride; D and Dv multiples of 8 up to 128)
+    → (out [T,Hq,Dv], lse [Hq,T]).  ``alibi_slopes`` fp32 [Hq]: adds ``slope_h · (key − query)`` to the scores;
+    ``sink`` fp32 [Hq]: one more term ``exp(sink_h)`` of the softmax denominator (part of lse)."""
     T, Hq, D = q.shape
-    Hk = k.shape[1]
+    Hk, Dv = k.shape[1], v.shape[2]
     for t, n in ((q, "q"), (k, "k"), (v, "v")):
-        if t.dtype != torch.bfloat16 or t.stride(2) != 1 or t.stride(1) != D:
-            raise ValueError(f"flash_attn_fwd: {n} must be bf16 with contiguous [heads, 128] rows")
-    if D != 128 or k.stride(0) != v.stride(0):
-        raise ValueError("flash_attn_fwd: head_dim must be 128 and k/v must share a row stride")
-    out = torch.empty(T, Hq, D, dtype=torch.bfloat16, device=q.device)
+        if t.dtype != torch.bfloat16 or t.stride(2) != 1 or (t.shape[1] > 1 and t.stride(1) != t.shape[2]):
+            raise ValueError(f"flash_attn_fwd: {n} must be bf16 with contiguous [heads, dim] rows")
+    if k.shape[2] != D or max(D, Dv) > 128 or D % 8 or Dv % 8:
+        raise ValueError("flash_attn_fwd: head sizes must be multiples of 8 up to 128, the same for q and k")
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != Hq or not sink.is_contiguous()):
+        raise ValueError("flash_attn_fwd: sink must be fp32 [heads]")
+    out = torch.empty(T, Hq, Dv, dtype=torch.bfloat16, device=q.device)
     lse = torch.empty(Hq, T, dtype=torch.float32, device=q.device)
     sl = _slopes(alibi_slopes, Hq, q.device)
     rc = lib().ell_flash_attn_fwd(_p(q), _p(k), _p(v), _p(out), _p(lse), _p(row_start), c_int(T), c_int(Hq), c_int(Hk),
-                                  c_int(q.stride(0)), c_int(k.stride(0)), c_float(scale), _p(sl),
-                                  _p(err_flag(q.device)), _stream())
+                                  c_int(D), c_int(Dv), c_int(q.stride(0)), c_int(k.stride(0)), c_int(v.stride(0)),
+                                  c_float(scale), _p(sl), _p(sink), _p(err_flag(q.device)), _stream())
     _check(rc, "flash_attn_fwd")
     return out, lse
 
