@@ -127,7 +127,15 @@ def main():
     ap.add_argument("--varlen", action="store_true",
                     help="packed variable-length documents (lengths uniform in [256, seq]) with cu_seqlens")
     ap.add_argument("--no-fused-tp", action="store_true", help="use the NCCL + GEMM composition for TP linears")
+    ap.add_argument("--serving", action="store_true", help="instead of the training step: prompt and decode throughput of "
+                    "the hybrid decoder beside a Llama of equal size (easyllm_b200/infer/bench_serving.py)")
+    ap.add_argument("--serving-sizes", default="2k,4k")
+    ap.add_argument("--serving-kernels", action="store_true", help="with --serving: also every kernel against its roofline")
     args = ap.parse_args()
+
+    if args.serving:
+        from easyllm_b200.infer import bench_serving
+        return bench_serving.main(args.serving_sizes.split(","), args.serving_kernels, clocks=lambda: ClockSampler(0))
 
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":

@@ -30,7 +30,7 @@ from ...ops import reference as ref
 from ..layers import RotaryTables, alibi_slopes
 from .feedforward import DenseGLU, SparseMoE
 from .mixers import ChannelDelta, DynamicTanh, TimeMix
-from .state import DecodeState, KVRows
+from .state import DecodeGraph, DecodeState, KVRows
 
 
 @dataclass
@@ -569,11 +569,12 @@ class CausalLM(nn.Module):
     @torch.no_grad()
     def _decode_steps(self, input_ids, max_new_tokens=64, do_sample=False, temperature=1.0, top_k=0, top_p=0.0,
                       eos_token_id=None, repetition_penalty=1.0, stop_words_ids=None, soft_prefix=None,
-                      attention_mask=None, **_):
+                      attention_mask=None, cuda_graph=True, **_):
         """Greedy / sampled decoding from the cache / state manager; yields the running ``[b, s]`` token tensor after
         every new token.  ``attention_mask``: rows of unequal length (padding on either side of ``input_ids``; new
         tokens are appended after column ``s``).  A row ends at ``eos_token_id`` or when its tail equals one of
         ``stop_words_ids`` (token sequences; the stop sequence stays in the output, later positions are filled with eos).
+        ``cuda_graph``: on a GPU, replay the decode step as a CUDA graph once it has run eagerly.
         ``soft_prefix``: ``{"embeds": [P, hidden]}`` (prompt tuning: virtual input embeddings in front of the
         prompt) or ``{"kv": [layers, 2, P, kv_heads, head_dim]}`` (prefix tuning: pre-filled cache entries)."""
         from ...infer.generation import sample_next
@@ -612,13 +613,19 @@ class CausalLM(nn.Module):
         seen_mask = real.to(dev)
         done = torch.zeros(b, dtype=torch.bool, device=dev)
         fill = eos if eos is not None else 0
+        graph = None
         for step in range(max_new_tokens):
             if step == 0:
                 h, meta = self.step(state, slots, prompts, inputs_embeds=embeds)
                 h = h[meta["last_rows"].to(h.device)]
+                logits = self.logits(h)
+            elif graph is not None:
+                logits = graph.step(toks[:, -1])
             else:
-                h, meta = self.step(state, slots, toks[:, -1])
-            logits = self.logits(h)
+                logits = self.logits(self.step(state, slots, toks[:, -1])[0])
+                if cuda_graph and dev.type == "cuda" and dt != torch.float16 and not a.use_cache_quantization and \
+                        max_new_tokens - step > 4:
+                    graph = DecodeGraph(self, state, slots)
             if repetition_penalty != 1.0:
                 seen = torch.gather(logits, 1, toks)
                 pen = torch.where(seen > 0, seen / repetition_penalty, seen * repetition_penalty)

@@ -9,8 +9,8 @@ layer contributes one state object through ``layer.new_state``:
 * a plain dict (the 8-bit cache of Qwen): dense batches of equal length only.
 
 ``DecodeState.step_meta`` is the packed description of one step that the layers read.  All index tensors are built on
-the host and copied once; a decode step (one token a sequence) of the same slots can be advanced in place on the
-device (``advance``), so its kernels can be replayed from a CUDA graph.
+the host and copied once; ``DecodeGraph`` replays the one-token step of fixed slots as a CUDA graph, with the positions
+advanced on the device.
 """
 from __future__ import annotations
 
@@ -93,7 +93,7 @@ class DecodeState:
         self.capacity = capacity
 
     # ---- one step ------------------------------------------------------------------------------
-    def step_meta(self, slots, counts):
+    def step_meta(self, slots, counts, advance=True):
         """Packed meta of a step that appends ``counts[i]`` tokens to ``slots[i]``; the lengths advance."""
         if len(set(slots)) != len(slots) or any(c < 1 for c in counts):
             raise ValueError("a step brings at least one token to each of its (distinct) sequences")
@@ -116,18 +116,41 @@ class DecodeState:
             buf = buf.pin_memory().to(dev, non_blocking=True)
         parts = buf.split([S + 1, S, S, T, T, T, T])
         for s, c in zip(slots, counts):
-            self.lengths[s] += c
+            self.lengths[s] += c if advance else 0
         fresh = not any(start)
         return {"cu_seqlens": parts[0], "seq_slot": parts[1], "seq_pos0": parts[2], "position_ids": parts[3],
                 "row_start": parts[4], "kv_base": parts[5], "kv_len": parts[6], "max_seqlen": max(counts),
                 "max_position": max(p + c for p, c in zip(start, counts)), "batch": S, "fresh": fresh,
                 "one_token": T == S, "kv_capacity": self.capacity,
-                "last_rows": torch.tensor(cu[1:]) - 1, "slots": list(slots)}
+                "last_rows": torch.tensor(cu[1:]) - 1}
 
-    def advance(self, meta):
-        """Turn the meta of a one-token step into that of the next one, on the device."""
-        for s in meta["slots"]:
-            self.lengths[s] += 1
-        meta["seq_pos0"].add_(1)
-        meta["position_ids"].add_(1)
-        meta["kv_len"].add_(1)
+
+class DecodeGraph:
+    """The one-token step of fixed slots as a CUDA graph: embedding, layers, logits and the advance of the positions,
+    replayed with new token ids.  The cache must not move while the graph is in use: its capacity is checked, and the
+    caller captures anew when the state has grown.  Capturing executes nothing, so no state is touched; run at least one
+    eager step before (it initialises the kernels)."""
+
+    def __init__(self, model, state, slots):
+        self.state, self.slots, self.capacity = state, list(slots), state.capacity
+        self.meta = state.step_meta(slots, [1] * len(slots), advance=False)
+        # host-side bounds that hold for every replay
+        self.meta.update(max_position=state.capacity, kv_bound=state.capacity, fresh=False, one_token=True)
+        self.ids = torch.zeros(len(slots), dtype=torch.long, device=state.device)
+        self.graph = torch.cuda.CUDAGraph()
+        torch.cuda.synchronize()
+        with torch.no_grad(), torch.cuda.graph(self.graph):
+            self.logits = model.logits(model.hidden_states(self.ids, self.meta, state.layers))
+            for name in ("seq_pos0", "position_ids", "kv_len"):
+                self.meta[name].add_(1)
+
+    def step(self, tokens):
+        """fp32 logits ``[n, vocab]`` after ``tokens [n]`` (a buffer the next step overwrites)."""
+        st = self.state
+        if st.capacity != self.capacity or any(st.lengths[s] >= self.capacity for s in self.slots):
+            raise RuntimeError("the cache moved or is full: capture the decode step again")
+        self.ids.copy_(tokens)
+        self.graph.replay()
+        for s in self.slots:
+            st.lengths[s] += 1
+        return self.logits

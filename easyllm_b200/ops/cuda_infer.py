@@ -116,7 +116,7 @@ def linear_add_(acc, x, w):
 
 # ---- elementwise -------------------------------------------------------------------------------
 def embed_scaled(ids, table, scale):
-    ids = ids.reshape(-1).to(torch.int64)
+    ids = ids.reshape(-1).to(torch.int64).contiguous()
     out = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
     _check(lib().ell_embed_scaled(_p(ids), _p(table), _p(out), c_int(ids.numel()), c_int(table.shape[1]),
                                   c_longlong(table.shape[0]), c_float(scale), _bf(table.dtype), _p(err_flag(table.device)),

@@ -225,6 +225,32 @@ def test_greedy_generation_of_an_unequal_batch(models, device):
         assert row[:cut] == full[:cut] and all(t == eos for t in row[cut:])
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("name", ["aligned", "wide"])
+def test_replayed_decode_steps_equal_eager_ones(models, name):
+    """The decode step as a CUDA graph, over the border of a cache tile, for an unequal batch."""
+    dev = _device("cuda")
+    cfg, w, model = models(name, dev, torch.bfloat16)
+    from easyllm_b200.models.hf_models.state import DecodeGraph
+    reqs = [pm.tokens(cfg, 90, 1), pm.tokens(cfg, 40, 2)]
+    logits = []
+    for replay in (False, True):
+        state = model.new_state(2, 128)
+        slots = [state.open(), state.open()]
+        run(model, state, slots, [r[:-35] for r in reqs])
+        graph, got = None, []
+        for i in range(35):
+            ids = torch.tensor([r[-35 + i] for r in reqs], device=dev)
+            if graph is not None:
+                got.append(graph.step(ids).clone())
+            else:
+                got.append(model.logits(model.step(state, slots, ids)[0]))
+                graph = DecodeGraph(model, state, slots) if replay else None
+        assert state.lengths[:2] == [90, 40] or state.lengths[slots[0]] == 90
+        logits.append(torch.stack(got))
+    assert error(logits[1].flatten(0, 1), logits[0].flatten(0, 1).double().cpu(), torch.bfloat16) < 1e-3
+
+
 def test_text_generation_entry_point(models):
     """The inference loop of the HF runner on a model from the registry."""
     from easyllm_b200.config.registry import MODULE_ZOO_REGISTRY
