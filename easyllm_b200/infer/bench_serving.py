@@ -122,12 +122,11 @@ def kernel_cases(s, T, B, context):
     for phase, n, m in (("prefill", T, meta(1, T)), ("prefill8", T, meta(8, T // 8)), ("decode", B, meta(B, 1))):
         ns = m["cu_seqlens"].numel() - 1
         x32, h = r(n, W, dtype=f32), r(n, W)
-        w1, b1 = r(W, dtype=f32), r(W, dtype=f32)
+        w1, b1, r_w = r(W, dtype=f32), r(W, dtype=f32), r(W)
         al = torch.tensor(0.5, device=dev)
         if phase != "prefill8":
             yield "dynamic_tanh", phase, lambda: ci.dynamic_tanh(x32, al, w1, b1, bf), 6 * n * W, 0, 0
             yield "llama rmsnorm+add", phase, lambda: cu.rmsnorm_fwd(h, h, r_w, 1e-6), 8 * n * W, 0, 0
-            r_w = r(W)
             gu = r(n, 2 * F)
             yield "glu gelu", phase, lambda: ci.glu(gu, "gelu_tanh"), 6 * n * F, 0, 0
             yield "llama swiglu", phase, lambda: cu.swiglu_fwd(gu), 6 * n * F, 0, 0

@@ -3,15 +3,16 @@
 //
 // Query row t sees the rows base[t] .. base[t] + len[t] - 1 of k [R, G, d] and v [R, G, dv] and sits at the last one.
 // A CTA of 128 threads takes (row t, kv head, a range of keys) with all `rep` query heads of that kv head (in groups of
-// at most 8), so every key and value is read once per group.  Tiles of 64 keys: eight lanes share a key for the scores
-// (16-byte loads, queries from shared memory), the softmax runs on the 64 scores of a head per warp, and the threads
-// own value columns for the weighted sum.  With more than one range per row a second kernel merges the partial
-// (max, sum, accumulator) triples; the sink joins the denominator at the end, once.
+// at most 8), so every key and value is read once per group.  Tiles of KT keys and values come through two
+// shared-memory stages (cp.async, the next tile in flight during the arithmetic).  Eight lanes share a key for the
+// scores, the softmax runs on the KT scores of a head per warp, and for the weighted sum a thread owns eight value
+// columns and a share of the tile's keys; the shares are added up once, at the end.  With more than one range per row a
+// second kernel merges the partial (max, sum, accumulator) triples; the sink joins the denominator at the end, once.
 #include "vec.cuh"
 
 namespace ell {
 
-constexpr int kArThreads = 128, kArKeys = 64, kArRep = 8;
+constexpr int kArThreads = 128, kArRep = 8;
 
 struct AttnRowsArgs {
   const void *q, *k, *v;
@@ -23,66 +24,119 @@ struct AttnRowsArgs {
   float scale;
 };
 
-template <typename T, bool VEC>
+// Shared memory: scaled queries [8][dp] | scores [8][KT] | statistics [8][4] | two stages of KT key rows, KT value rows.
+struct ArLayout {
+  int dp, krow, vrow, kgroups;    // padded key size; row strides in elements; key shares of the weighted sum
+  int stage, bytes;               // elements of a stage; total bytes
+};
+__host__ __device__ inline ArLayout ar_layout(int d, int dv, int esz, int KT) {
+  ArLayout l;
+  l.dp = (d + 63) / 64 * 64;
+  l.krow = l.dp + 16 / esz;
+  const int oct = (dv + 7) / 8;
+  l.vrow = oct * 8 + 16 / esz;
+  l.kgroups = 1;
+  while (2 * l.kgroups * oct <= kArThreads && 2 * l.kgroups <= KT / 4 && l.kgroups < 16) l.kgroups *= 2;
+  l.stage = KT * (l.krow + l.vrow);
+  const int head = (kArRep * l.dp + kArRep * KT + kArRep * 4) * 4;
+  const int a = 2 * l.stage * esz, b = l.kgroups * kArRep * oct * 8 * 4;   // the sums reuse the stages
+  l.bytes = head + (a > b ? a : b);
+  return l;
+}
+
+template <typename T, int KT, bool VEC>
 __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArgs a) {
-  extern __shared__ float sm[];
+  extern __shared__ __align__(16) float sm[];
+  const ArLayout L = ar_layout(a.d, a.dv, sizeof(T), KT);
   const int t = blockIdx.x, rep = a.H / a.G, groups = (rep + kArRep - 1) / kArRep;
   const int g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * kArRep;
   const int nh = min(kArRep, g * rep + rep - h0);
-  const int split = blockIdx.z;
-  const int dp = (a.d + 63) / 64 * 64;
-  float* qs = sm;                                   // [nh][dp]
-  float* p = qs + kArRep * dp;                      // [nh][kArKeys]
-  float* stat = p + kArRep * kArKeys;               // [nh][4]: max, sum, rescale
+  const int split = blockIdx.z, dp = L.dp, oct = (a.dv + 7) / 8;
+  float* qs = sm;
+  float* p = qs + kArRep * dp;
+  float* stat = p + kArRep * KT;                    // max, sum, rescale
+  T* stages = reinterpret_cast<T*>(stat + kArRep * 4);
   const int len = a.len[t];
   const size_t base = a.base[t];
   const int k0 = split * a.range, k1 = min(k0 + a.range, len);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int i = threadIdx.x; i < nh * dp; i += kArThreads) {
+  // rows and columns the copies leave out must read as zero
+  for (int i = threadIdx.x; i < 2 * L.stage * (int)sizeof(T) / 16; i += kArThreads)
+    reinterpret_cast<uint4*>(stages)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = threadIdx.x; i < kArRep * dp; i += kArThreads) {
     const int h = i / dp, c = i % dp;
-    qs[i] = c < a.d ? to_f<T>(reinterpret_cast<const T*>(a.q)[(size_t)t * a.ldq + (size_t)(h0 + h) * a.d + c]) * a.scale : 0.f;
+    qs[i] = h < nh && c < a.d
+                ? to_f<T>(reinterpret_cast<const T*>(a.q)[(size_t)t * a.ldq + (size_t)(h0 + h) * a.d + c]) * a.scale : 0.f;
   }
-  if (threadIdx.x < nh) {
+  if (threadIdx.x < kArRep) {
     stat[threadIdx.x * 4] = -INFINITY;
     stat[threadIdx.x * 4 + 1] = 0.f;
   }
-  // value columns of this thread: c = threadIdx.x + 128 j, up to 4 per pass (dv <= 512)
-  float acc[kArRep][4];
-#pragma unroll
-  for (int h = 0; h < kArRep; ++h)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) acc[h][j] = 0.f;
   __syncthreads();
   const T* kb = reinterpret_cast<const T*>(a.k) + base * a.ldk + (size_t)g * a.d;
   const T* vb = reinterpret_cast<const T*>(a.v) + base * a.ldv + (size_t)g * a.dv;
+  auto load_tile = [&](int kt, int buf) {
+    T* ks = stages + buf * L.stage;
+    T* vs = ks + KT * L.krow;
+    const int cnt = min(KT, k1 - kt);
+    if (VEC) {
+      constexpr int per = 16 / sizeof(T);
+      const int kp = a.d / per, vp = a.dv / per;
+      for (int i = threadIdx.x; i < cnt * kp; i += kArThreads) {
+        const int r = i / kp, c = (i % kp) * per;
+        cp_async16(ks + r * L.krow + c, kb + (size_t)(kt + r) * a.ldk + c);
+      }
+      for (int i = threadIdx.x; i < cnt * vp; i += kArThreads) {
+        const int r = i / vp, c = (i % vp) * per;
+        cp_async16(vs + r * L.vrow + c, vb + (size_t)(kt + r) * a.ldv + c);
+      }
+    } else {
+      for (int i = threadIdx.x; i < cnt * a.d; i += kArThreads)
+        ks[i / a.d * L.krow + i % a.d] = kb[(size_t)(kt + i / a.d) * a.ldk + i % a.d];
+      for (int i = threadIdx.x; i < cnt * a.dv; i += kArThreads)
+        vs[i / a.dv * L.vrow + i % a.dv] = vb[(size_t)(kt + i / a.dv) * a.ldv + i % a.dv];
+    }
+    cp_async_commit();
+  };
+  // weighted sum: this thread's eight columns and its share of a tile's keys
+  const int my_oct = threadIdx.x % oct, my_share = threadIdx.x / oct, share = KT / L.kgroups;
+  const bool adds = my_share < L.kgroups;
+  float acc[kArRep][8];
+#pragma unroll
+  for (int h = 0; h < kArRep; ++h)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[h][j] = 0.f;
   const int l8 = lane & 7, grp = warp * 4 + (lane >> 3);          // 16 groups of 8 lanes
-  for (int kt = k0; kt < k1; kt += kArKeys) {
-    // scores: group takes keys grp, grp + 16, grp + 32, grp + 48 of the tile
-    float sc[kArRep][4];
+  constexpr int KJ = KT / 16;
+  if (k0 < k1) load_tile(k0, 0);
+  int buf = 0;
+  for (int kt = k0; kt < k1; kt += KT, buf ^= 1) {
+    if (kt + KT < k1) {
+      load_tile(kt + KT, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const T* ks = stages + buf * L.stage;
+    const T* vs = ks + KT * L.krow;
+    // scores: a group takes keys grp, grp + 16, ...
+    float sc[kArRep][KJ];
 #pragma unroll
     for (int h = 0; h < kArRep; ++h)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) sc[h][j] = 0.f;
+      for (int j = 0; j < KJ; ++j) sc[h][j] = 0.f;
     for (int c = l8 * 8; c < dp; c += 64) {
-      float kv[4][8];
+      float kv[KJ][8];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int key = kt + grp + 16 * j;
-        const T* kp = kb + (size_t)key * a.ldk + c;
-        if (key < k1 && VEC && c + 7 < a.d) {
-          load_v<8>(kp, kv[j]);
-        } else {
-#pragma unroll
-          for (int i = 0; i < 8; ++i) kv[j][i] = key < k1 && c + i < a.d ? to_f<T>(kp[i]) : 0.f;
-        }
-      }
+      for (int j = 0; j < KJ; ++j) load_v<8>(ks + (grp + 16 * j) * L.krow + c, kv[j]);
 #pragma unroll
       for (int h = 0; h < kArRep; ++h) {
         if (h < nh) {
           const float4 q0 = *reinterpret_cast<const float4*>(qs + h * dp + c);
           const float4 q1 = *reinterpret_cast<const float4*>(qs + h * dp + c + 4);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
+          for (int j = 0; j < KJ; ++j) {
             float s = sc[h][j];
             s = fmaf(q0.x, kv[j][0], s); s = fmaf(q0.y, kv[j][1], s); s = fmaf(q0.z, kv[j][2], s); s = fmaf(q0.w, kv[j][3], s);
             s = fmaf(q1.x, kv[j][4], s); s = fmaf(q1.y, kv[j][5], s); s = fmaf(q1.z, kv[j][6], s); s = fmaf(q1.w, kv[j][7], s);
@@ -95,7 +149,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
     for (int h = 0; h < kArRep; ++h) {
       if (h < nh) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < KJ; ++j) {
           float s = sc[h][j];
           s += __shfl_xor_sync(0xffffffffu, s, 1);
           s += __shfl_xor_sync(0xffffffffu, s, 2);
@@ -103,19 +157,28 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
           const int key = kt + grp + 16 * j;
           if (l8 == 0) {
             if (a.slopes != nullptr) s += a.slopes[h0 + h] * (float)(key - (len - 1));
-            p[h * kArKeys + grp + 16 * j] = key < k1 ? s : -INFINITY;
+            p[h * KT + grp + 16 * j] = key < k1 ? s : -INFINITY;
           }
         }
       }
     }
     __syncthreads();
     for (int h = warp; h < nh; h += 4) {
-      const float s0 = p[h * kArKeys + lane], s1 = p[h * kArKeys + 32 + lane];
-      const float m_old = stat[h * 4], m = fmaxf(m_old, warp_max(fmaxf(s0, s1)));   // finite: the tile has a key
-      const float e0 = expf(s0 - m), e1 = expf(s1 - m);
-      p[h * kArKeys + lane] = e0;
-      p[h * kArKeys + 32 + lane] = e1;
-      const float sum = warp_sum(e0 + e1);
+      float s[(KT + 31) / 32], mx = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < (KT + 31) / 32; ++j) {
+        s[j] = 32 * j + lane < KT ? p[h * KT + 32 * j + lane] : -INFINITY;
+        mx = fmaxf(mx, s[j]);
+      }
+      const float m_old = stat[h * 4], m = fmaxf(m_old, warp_max(mx));   // finite: the tile has a key
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < (KT + 31) / 32; ++j) {
+        const float e = expf(s[j] - m);
+        sum += e;
+        if (32 * j + lane < KT) p[h * KT + 32 * j + lane] = e;
+      }
+      sum = warp_sum(sum);
       if (lane == 0) {
         const float al = expf(m_old - m);
         stat[h * 4] = m;
@@ -124,48 +187,47 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
       }
     }
     __syncthreads();
-    const int cnt = min(kArKeys, k1 - kt);
+    if (adds) {
 #pragma unroll
-    for (int h = 0; h < kArRep; ++h) {
-      if (h < nh) {
-        const float al = stat[h * 4 + 2];
+      for (int h = 0; h < kArRep; ++h) {
+        if (h < nh) {
+          const float al = stat[h * 4 + 2];
+          if (al != 1.f) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[h][j] *= al;
-      }
-    }
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int c = threadIdx.x + kArThreads * j;
-      if (c < a.dv) {
-        const T* vp = vb + (size_t)kt * a.ldv + c;
-        int i = 0;
-        for (; i + 4 <= cnt; i += 4) {
-          float vv[4];
-#pragma unroll
-          for (int x = 0; x < 4; ++x) vv[x] = to_f<T>(vp[(size_t)(i + x) * a.ldv]);
-#pragma unroll
-          for (int h = 0; h < kArRep; ++h) {
-            if (h < nh) {
-              const float4 w = *reinterpret_cast<const float4*>(p + h * kArKeys + i);
-              acc[h][j] = fmaf(w.x, vv[0], acc[h][j]); acc[h][j] = fmaf(w.y, vv[1], acc[h][j]);
-              acc[h][j] = fmaf(w.z, vv[2], acc[h][j]); acc[h][j] = fmaf(w.w, vv[3], acc[h][j]);
-            }
+            for (int j = 0; j < 8; ++j) acc[h][j] *= al;
           }
         }
-        for (; i < cnt; ++i) {
-          const float vv = to_f<T>(vp[(size_t)i * a.ldv]);
+      }
+      const T* vp = vs + (size_t)(my_share * share) * L.vrow + my_oct * 8;
+      for (int i = 0; i < share; i += 4) {
+        float vv[4][8];
 #pragma unroll
-          for (int h = 0; h < kArRep; ++h)
-            if (h < nh) acc[h][j] = fmaf(p[h * kArKeys + i], vv, acc[h][j]);
+        for (int x = 0; x < 4; ++x) load_v<8>(vp + (i + x) * L.vrow, vv[x]);
+#pragma unroll
+        for (int h = 0; h < kArRep; ++h) {
+          if (h < nh) {
+            const float4 w = *reinterpret_cast<const float4*>(p + h * KT + my_share * share + i);
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              acc[h][j] = fmaf(w.w, vv[3][j], fmaf(w.z, vv[2][j], fmaf(w.y, vv[1][j], fmaf(w.x, vv[0][j], acc[h][j]))));
+          }
         }
       }
     }
     __syncthreads();
   }
-  // results
+  // add the shares up: sums[share][head][column] over the stages' memory
+  float* sums = reinterpret_cast<float*>(stages);
+  if (adds) {
 #pragma unroll
-  for (int h = 0; h < kArRep; ++h) {
-    if (h >= nh) continue;
+    for (int h = 0; h < kArRep; ++h)
+      if (h < nh) store_v<8>(sums + ((my_share * kArRep + h) * oct + my_oct) * 8, acc[h]);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * a.dv; i += kArThreads) {
+    const int h = i / a.dv, c = i % a.dv;
+    float o = 0.f;
+    for (int x = 0; x < L.kgroups; ++x) o += sums[(x * kArRep + h) * oct * 8 + c];
     const float m = stat[h * 4], l = stat[h * 4 + 1];
     if (a.splits == 1) {
       float den = l, f = 1.f;
@@ -174,22 +236,14 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
         f = expf(m - mm);
         den = l * f + expf(sk - mm);
       }
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = threadIdx.x + kArThreads * j;
-        if (c < a.dv) reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h0 + h) * a.dv + c] = from_f<T>(acc[h][j] * f / den);
-      }
+      reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h0 + h) * a.dv + c] = from_f<T>(o * f / den);
     } else {
       float* pt = a.part + (((size_t)t * a.H + h0 + h) * a.splits + split) * (a.dv + 2);
-      if (threadIdx.x == 0) {
+      if (c == 0) {
         pt[0] = m;
         pt[1] = l;
       }
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = threadIdx.x + kArThreads * j;
-        if (c < a.dv) pt[2 + c] = acc[h][j];
-      }
+      pt[2 + c] = o;
     }
   }
 }
@@ -211,15 +265,37 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_merge_kernel(const AttnR
   }
 }
 
-// Ranges per row: enough CTAs to fill the GPU a few times, at least 128 keys each.
+// Ranges per row: enough CTAs to fill the GPU a few times, about 256 keys each at least.
 static int attn_rows_splits(int n, int H, int G, int max_len) {
   const int rep = H / G;
   const long long ctas = (long long)n * G * ((rep + kArRep - 1) / kArRep);
   long long s = (4LL * kNumSMs + ctas - 1) / ctas;
-  const long long most = (max_len + 127) / 128;
+  const long long most = (max_len + 255) / 256;
   if (s > most) s = most;
   if (s > 64) s = 64;
   return s < 1 ? 1 : (int)s;
+}
+
+template <typename T, int KT, bool VEC>
+static int launch_attn_rows_kt(const AttnRowsArgs& a, dim3 grid, cudaStream_t stream) {
+  const int bytes = ar_layout(a.d, a.dv, sizeof(T), KT).bytes;
+  auto kern = attn_rows_kernel<T, KT, VEC>;
+  static int configured = 0;
+  if (bytes > configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return (int)e;
+    configured = bytes;
+  }
+  kern<<<grid, kArThreads, bytes, stream>>>(a);
+  if (a.splits > 1) attn_rows_merge_kernel<T><<<dim3(a.n, a.H), kArThreads, 0, stream>>>(a);
+  return launch_status();
+}
+
+template <typename T>
+static int launch_attn_rows(const AttnRowsArgs& a, dim3 grid, bool vec, cudaStream_t stream) {
+  const bool small = ar_layout(a.d, a.dv, sizeof(T), 64).bytes > 160 * 1024;      // very wide fp32 heads: short tiles
+  if (small) return vec ? launch_attn_rows_kt<T, 16, true>(a, grid, stream) : launch_attn_rows_kt<T, 16, false>(a, grid, stream);
+  return vec ? launch_attn_rows_kt<T, 64, true>(a, grid, stream) : launch_attn_rows_kt<T, 64, false>(a, grid, stream);
 }
 
 }  // namespace ell
@@ -237,24 +313,15 @@ ELL_API int ell_attn_rows(const void* q, const void* k, const void* v, void* out
                           const int* len, const float* sink, const float* slopes, int n, int H, int G, int d, int dv,
                           int ldq, int ldk, int ldv, int max_len, float scale, int is_bf16, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (H % G || dv > 4 * kArThreads || d > 512 || H > 65535) return -2;
+  if (H % G || dv > 512 || d > 512 || H > 65535) return -2;
   AttnRowsArgs a{q, k, v, out, part, base, len, sink, slopes, n, H, G, d, dv, ldq, ldk, ldv, 1, 0, scale};
   a.splits = attn_rows_splits(n, H, G, max_len);
-  a.range = ((max_len + a.splits - 1) / a.splits + kArKeys - 1) / kArKeys * kArKeys;
+  a.range = ((max_len + a.splits - 1) / a.splits + 63) / 64 * 64;
   if (a.splits > 1 && part == nullptr) return -2;
-  const int rep = H / G, dp = (d + 63) / 64 * 64;
-  const size_t smem = (size_t)(kArRep * dp + kArRep * kArKeys + kArRep * 4) * 4;
+  const int rep = H / G;
   dim3 grid(n, G * ((rep + kArRep - 1) / kArRep), a.splits);
   const int esz = is_bf16 ? 2 : 4;
-  const bool vec = d % 8 == 0 && (ldk * esz) % 16 == 0 && aligned_to(k, 16);
-  if (is_bf16) {
-    if (vec) attn_rows_kernel<__nv_bfloat16, true><<<grid, kArThreads, smem, stream>>>(a);
-    else attn_rows_kernel<__nv_bfloat16, false><<<grid, kArThreads, smem, stream>>>(a);
-    if (a.splits > 1) attn_rows_merge_kernel<__nv_bfloat16><<<dim3(n, H), kArThreads, 0, stream>>>(a);
-  } else {
-    if (vec) attn_rows_kernel<float, true><<<grid, kArThreads, smem, stream>>>(a);
-    else attn_rows_kernel<float, false><<<grid, kArThreads, smem, stream>>>(a);
-    if (a.splits > 1) attn_rows_merge_kernel<float><<<dim3(n, H), kArThreads, 0, stream>>>(a);
-  }
-  return launch_status();
+  const bool vec = (d * esz) % 16 == 0 && (dv * esz) % 16 == 0 && (ldk * esz) % 16 == 0 && (ldv * esz) % 16 == 0 &&
+                   aligned_to(k, 16) && aligned_to(v, 16);
+  return is_bf16 ? launch_attn_rows<__nv_bfloat16>(a, grid, vec, stream) : launch_attn_rows<float>(a, grid, vec, stream);
 }

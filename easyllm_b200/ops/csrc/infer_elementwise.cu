@@ -147,15 +147,42 @@ __global__ void token_mix_kernel(const T* __restrict__ h, const float* __restric
   }
 }
 
-// One warp per (token, head): y = o / rms(o) * w * act(gate).
-template <typename T, int V>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate,
-                                      T* __restrict__ y, int n, int H, int dv, int w_per_head, int ldg, int silu_gate,
-                                      float eps) {
-  const int warps = blockDim.x >> 5, lane = threadIdx.x & 31;
-  for (long long i = blockIdx.x * (long long)warps + (threadIdx.x >> 5); i < (long long)n * H; i += (long long)gridDim.x * warps) {
-    const int t = (int)(i / H), hd = (int)(i % H);
-    const float* orow = o + (size_t)i * dv;
+// One warp per (token, head): y = o / rms(o) * w * act(gate).  IT pieces of V elements a lane are kept in registers, all
+// loads ahead of the reduction (IT = 0: any head size, read twice).
+template <typename T, int V, int IT>
+__device__ __forceinline__ void head_norm_gate_row(const float* orow, const float* w, const T* gate, T* y, int dv,
+                                                   int silu_gate, float eps, int lane) {
+  if (IT > 0) {
+    float f[IT > 0 ? IT : 1][V], g[IT > 0 ? IT : 1][V];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int c = (i * 32 + lane) * V;
+      if (c < dv) {
+        load_v<V>(orow + c, f[i]);
+        load_v<V>(gate + c, g[i]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[i][j] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < IT; ++i)
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += f[i][j] * f[i][j];
+    const float r = 1.f / sqrtf(warp_sum(ss) / dv + eps);
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int c = (i * 32 + lane) * V;
+      if (c < dv) {
+        float wv[V];
+        load_v<V>(w + c, wv);
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[i][j] = f[i][j] * r * wv[j] * (silu_gate ? silu_f(g[i][j]) : sigmoid_f(g[i][j]));
+        store_v<V>(y + c, f[i]);
+      }
+    }
+  } else {
     float ss = 0.f;
     for (int c = lane * V; c < dv; c += 32 * V) {
       float f[V];
@@ -167,12 +194,29 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
     for (int c = lane * V; c < dv; c += 32 * V) {
       float f[V], g[V], wv[V];
       load_v<V>(orow + c, f);
-      load_v<V>(gate + (size_t)t * ldg + (size_t)hd * dv + c, g);
-      load_v<V>(w + (w_per_head ? hd * dv : 0) + c, wv);
+      load_v<V>(gate + c, g);
+      load_v<V>(w + c, wv);
 #pragma unroll
       for (int j = 0; j < V; ++j) f[j] = f[j] * r * wv[j] * (silu_gate ? silu_f(g[j]) : sigmoid_f(g[j]));
-      store_v<V>(y + (size_t)i * dv + c, f);
+      store_v<V>(y + c, f);
     }
+  }
+}
+
+template <typename T, int V>
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate,
+                                      T* __restrict__ y, int n, int H, int dv, int w_per_head, int ldg, int silu_gate,
+                                      float eps) {
+  const int warps = blockDim.x >> 5, lane = threadIdx.x & 31;
+  for (long long i = blockIdx.x * (long long)warps + (threadIdx.x >> 5); i < (long long)n * H; i += (long long)gridDim.x * warps) {
+    const int t = (int)(i / H), hd = (int)(i % H);
+    const float* orow = o + (size_t)i * dv;
+    const float* wrow = w + (w_per_head ? hd * dv : 0);
+    const T* grow = gate + (size_t)t * ldg + (size_t)hd * dv;
+    T* yrow = y + (size_t)i * dv;
+    if (V == 4 && dv <= 128) head_norm_gate_row<T, V, 1>(orow, wrow, grow, yrow, dv, silu_gate, eps, lane);
+    else if (V == 4 && dv <= 256) head_norm_gate_row<T, V, 2>(orow, wrow, grow, yrow, dv, silu_gate, eps, lane);
+    else head_norm_gate_row<T, V, 0>(orow, wrow, grow, yrow, dv, silu_gate, eps, lane);
   }
 }
 
@@ -285,7 +329,7 @@ ELL_API int ell_head_norm_gate(const float* o, const float* w, const void* gate,
   if (n <= 0) return 0;
   const bool v = dv % 4 == 0 && ldg % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 16) && aligned_to(gate, 16) &&
                  aligned_to(y, 16);
-  const int g = grid_for((long long)n * H, 8);
+  const int g = grid_for((long long)n * H, 8, 64);
   ELL_TV(v, head_norm_gate_kernel, g, 256, o, w, (const T*)gate, (T*)y, n, H, dv, w_per_head, ldg, silu_gate, eps);
   return launch_status();
 }

@@ -1,7 +1,10 @@
 // y = x · Wᵀ for a few rows of x (decoding) and for row lengths the TMA-fed GEMM cannot take: bound by the weight bytes.
 //
-// A warp computes NW rows of W against MR rows of x: lanes stride over K with 16-byte loads of W (bf16) and of x (L1),
-// fp32 accumulation, one shuffle reduction per result.  KS warps of a CTA may split K when N alone gives too few warps.
+// bf16: a warp multiplies 16 rows of W with up to 16 rows of x on mma.sync m16n8k16 (the products are few, the point is
+// to keep the instruction count far below the load rate): a thread loads 8 consecutive k of a row with one 16-byte load
+// and feeds them to two instructions, in an order of k that is the same for both operands.  The warps of a CTA split K.
+// fp32, and shapes without 16-byte rows: a warp computes NW rows of W against MR rows of x, lanes striding over K, fp32
+// fused multiply-adds, one shuffle reduction per result.
 // Optional bias, tanh, fp32 output, or accumulation into an fp32 matrix; a batch of equally shaped products in grid.z.
 #include "vec.cuh"
 
@@ -79,6 +82,91 @@ __global__ void __launch_bounds__(kMvWarps * 32) matvec_kernel(const MatvecArgs 
     else if (a.out_f32) reinterpret_cast<float*>(a.out)[o] = v;
     else reinterpret_cast<T*>(a.out)[o] = from_f<T>(v);
   }
+}
+
+__device__ __forceinline__ void mma_16816(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// MT tiles of 8 rows of x.  Rows of W and of x past the end are clamped (their results are dropped); k past the end is
+// clamped too, with x taken as zero.
+template <int MT>
+__global__ void __launch_bounds__(kMvWarps * 32) matvec_mma_kernel(const MatvecArgs a) {
+  __shared__ float red[kMvWarps][16][8 * MT + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int ks = a.ks, part = warp % ks, n0 = (blockIdx.x * (kMvWarps / ks) + warp / ks) * 16;
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + blockIdx.z * a.xb;
+  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.w) + blockIdx.z * a.wb;
+  const __nv_bfloat16* w0 = w + (size_t)min(n0 + g, a.N - 1) * a.K;
+  const __nv_bfloat16* w1 = w + (size_t)min(n0 + g + 8, a.N - 1) * a.K;
+  const __nv_bfloat16* xr[MT];
+#pragma unroll
+  for (int m = 0; m < MT; ++m) xr[m] = x + (size_t)min(m * 8 + g, a.M - 1) * a.ldx;
+  float c0[MT][4], c1[MT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) c0[m][i] = c1[m][i] = 0.f;
+  constexpr int U = 4;
+  const int nkb = (a.K + 31) / 32;
+  for (int kb = part; kb < nkb; kb += ks * U) {
+    uint4 wa[U], wb[U], xv[U][MT];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = (kb + u * ks) * 32 + t * 8;
+      const bool in = k < a.K;
+      const int kc = in ? k : 0;
+      wa[u] = *reinterpret_cast<const uint4*>(w0 + kc);
+      wb[u] = *reinterpret_cast<const uint4*>(w1 + kc);
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        xv[u][m] = *reinterpret_cast<const uint4*>(xr[m] + kc);
+        if (!in) xv[u][m] = make_uint4(0, 0, 0, 0);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        mma_16816(c0[m], wa[u].x, wb[u].x, wa[u].y, wb[u].y, xv[u][m].x, xv[u][m].y);
+        mma_16816(c1[m], wa[u].z, wb[u].z, wa[u].w, wb[u].w, xv[u][m].z, xv[u][m].w);
+      }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
+    red[warp][g][m * 8 + 2 * t] = c0[m][0] + c1[m][0];
+    red[warp][g][m * 8 + 2 * t + 1] = c0[m][1] + c1[m][1];
+    red[warp][g + 8][m * 8 + 2 * t] = c0[m][2] + c1[m][2];
+    red[warp][g + 8][m * 8 + 2 * t + 1] = c0[m][3] + c1[m][3];
+  }
+  __syncthreads();
+  const int rows = (kMvWarps / ks) * 16;
+  for (int e = threadIdx.x; e < rows * 8 * MT; e += kMvWarps * 32) {
+    const int r = e % rows, m = e / rows, n = blockIdx.x * rows + r;
+    if (n >= a.N || m >= a.M) continue;
+    float v = 0.f;
+    for (int p = 0; p < ks; ++p) v += red[(r >> 4) * ks + p][r & 15][m];
+    if (a.bias != nullptr) v += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.bias)[n]);
+    if (a.act_tanh) v = tanhf(v);
+    const size_t o = blockIdx.z * a.ob + (size_t)m * a.ldo + n;
+    if (a.accumulate) reinterpret_cast<float*>(a.out)[o] += v;
+    else if (a.out_f32) reinterpret_cast<float*>(a.out)[o] = v;
+    else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16_rn(v);
+  }
+}
+
+static int launch_matvec_mma(MatvecArgs a, int batch, cudaStream_t stream) {
+  const int nkb = (a.K + 31) / 32, tiles = (a.N + 15) / 16;
+  a.ks = kMvWarps;
+  while (a.ks > 1 && (nkb < 4 * a.ks || (long long)tiles * batch * a.ks > 64LL * kNumSMs)) a.ks /= 2;
+  const int per = kMvWarps / a.ks;
+  dim3 grid((tiles + per - 1) / per, 1, batch);
+  if (a.M <= 8) matvec_mma_kernel<1><<<grid, kMvWarps * 32, 0, stream>>>(a);
+  else matvec_mma_kernel<2><<<grid, kMvWarps * 32, 0, stream>>>(a);
+  return launch_status();
 }
 
 template <typename T, int MR, int NW>
@@ -308,6 +396,7 @@ ELL_API int ell_matvec(const void* x, const void* w, const void* bias, void* out
   const int esz = is_bf16 ? 2 : 4;
   const bool vec = K % 8 == 0 && (ldx * esz) % 16 == 0 && aligned_to(x, 16) && aligned_to(w, 16) && (xb * esz) % 16 == 0 &&
                    (wb * esz) % 16 == 0;
+  if (is_bf16 && vec && M <= 16) return launch_matvec_mma(a, batch, stream);
   return is_bf16 ? dispatch_matvec<__nv_bfloat16>(a, batch, vec, stream) : dispatch_matvec<float>(a, batch, vec, stream);
 }
 

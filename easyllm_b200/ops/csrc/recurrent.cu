@@ -9,14 +9,16 @@
 // keeps rows 32 i + 4 r .. + 3 in registers for the whole sequence.  Both sums of the delta rule are taken from the
 // decayed state at once (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the
 // token-to-token chain.
-// Warps 0-7 run the recurrence; warps 8-11 stage the next tokens' operands in shared memory (two buffers), compute the
+// Warps 0-7 run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Warps 8-11 copy the operands of the coming tokens
+// into a ring of shared-memory stages with cp.async (three stages ahead), convert bf16 operands to fp32, compute the
 // per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous tokens' outputs.
 #include "vec.cuh"
 
 namespace ell {
 
 constexpr int kScanCols = 32;         // value columns of a CTA
-constexpr int kScanTok = 16;          // tokens per stage
+constexpr int kScanTok = 8;           // tokens per stage (one per lane of a column's group: see the outputs)
+constexpr int kScanRing = 4;
 constexpr int kScanWarps = 8, kLoadWarps = 4;
 constexpr int kScanThreads = (kScanWarps + kLoadWarps) * 32;
 
@@ -33,26 +35,64 @@ struct ScanArgs {
   int H, G, d, dv, ldq, ldk, ldv;   // row strides of q, k, v in elements
 };
 
+// packed pairs of fp32
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float sum2(f32x2 a) {
+  float lo, hi;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a));
+  return lo + hi;
+}
+
+// One warp copies n elements; vec: 16-byte pieces (start and length multiples of 16 bytes), else 4-byte ones (fp32).
 template <typename T>
-__device__ __forceinline__ float4 load4_guard(const T* p, int c, int d, bool vec) {
-  float f[4] = {0.f, 0.f, 0.f, 0.f};
-  if (vec && c + 3 < d) {
-    load_v<4>(p + c, f);
-  } else {
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-      if (c + j < d) f[j] = to_f<T>(p[c + j]);
+__device__ __forceinline__ void warp_copy(T* dst, const T* src, int n, bool vec, int lane) {
+  if (vec) {
+    constexpr int kPer = 16 / sizeof(T);
+    for (int c = lane * kPer; c < n; c += 32 * kPer) cp_async16(dst + c, src + c);
+  } else if (sizeof(T) == 4) {
+    for (int c = lane; c < n; c += 32) cp_async4(dst + c, src + c);
   }
-  return make_float4(f[0], f[1], f[2], f[3]);
+}
+
+// Token record the recurrence reads: q | k | g | v | scalar, beta (fp32).  Raw bf16 record: g | beta (fp32), q | k | v.
+template <int NI>
+struct ScanTok {
+  static constexpr int kDp = NI * 32;
+  static constexpr int kFloats = 3 * kDp + kScanCols + 4;
+  static constexpr int kRawBytes = (kDp + 4) * 4 + (2 * kDp + kScanCols) * 2;
+};
+template <typename T, int NI>
+__host__ __device__ constexpr int scan_smem_bytes() {
+  using R = ScanTok<NI>;
+  const int out = 2 * kScanTok * kScanCols * 4;
+  return sizeof(T) == 4 ? kScanRing * kScanTok * R::kFloats * 4 + out
+                        : 2 * kScanTok * R::kFloats * 4 + kScanRing * kScanTok * R::kRawBytes + out;
 }
 
 template <int MODE, typename T, int NI>
 __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, int vec) {
-  constexpr int DP = NI * 32;
-  constexpr int kTokFloats = 3 * DP + kScanCols + 4;   // q | k | g | v | scalar, beta
-  extern __shared__ float sm[];
-  float* stage[2] = {sm, sm + kScanTok * kTokFloats};
-  float* outb = sm + 2 * kScanTok * kTokFloats;        // [2][kScanTok][kScanCols]
+  using R = ScanTok<NI>;
+  constexpr int DP = R::kDp, TF = R::kFloats;
+  constexpr bool kF32 = sizeof(T) == 4;
+  constexpr int kBufs = kF32 ? kScanRing : 2;          // fp32 records: the ring itself, or two converted stages
+  extern __shared__ __align__(16) float sm[];
+  float* outb = sm + kBufs * kScanTok * TF;            // [2][kScanTok][kScanCols]
+  uint8_t* raw = reinterpret_cast<uint8_t*>(outb + 2 * kScanTok * kScanCols);
   const int s = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * kScanCols;
   const int t_begin = a.cu[s], n_tok = a.cu[s + 1] - t_begin;
   if (n_tok <= 0) return;
@@ -65,141 +105,188 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
   const int col = col0 + cl;
   const bool live = !loader && col < a.dv;
 
-  auto load_chunk = [&](int ch) {
-    float* st = stage[ch & 1];
-    const int cnt = min(kScanTok, n_tok - ch * kScanTok);
-    for (int i = warp - kScanWarps; i < cnt; i += kLoadWarps) {
-      const size_t t = (size_t)t_begin + ch * kScanTok + i;
-      float* tok = st + i * kTokFloats;
-      const T* qp = reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
-      const T* kp = reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
-      const float* gp = a.g + (t * a.H + h) * a.d;
-      float dot = 0.f;
-#pragma unroll
-      for (int c0 = 0; c0 < DP; c0 += 128) {
-        const int c = c0 + lane * 4;
-        if (c < DP) {
-          const float4 q = load4_guard<T>(qp, c, a.d, vec), k = load4_guard<T>(kp, c, a.d, vec);
-          const float4 g = load4_guard<float>(gp, c, a.d, vec);
-          *reinterpret_cast<float4*>(tok + c) = q;
-          *reinterpret_cast<float4*>(tok + DP + c) = k;
-          *reinterpret_cast<float4*>(tok + 2 * DP + c) = g;
-          if (MODE == kWkv) {
-            const float4 u = load4_guard<float>(a.u + (size_t)h * a.d, c, a.d, vec);
-            dot += q.x * k.x * u.x + q.y * k.y * u.y + q.z * k.z * u.z + q.w * k.w * u.w;
-          } else {
-            dot += q.x * k.x + q.y * k.y + q.z * k.z + q.w * k.w;
-          }
-        }
-      }
-      const int c = col0 + lane;
-      tok[3 * DP + lane] = c < a.dv ? to_f<T>(reinterpret_cast<const T*>(a.v)[t * a.ldv + (size_t)h * a.dv + c]) : 0.f;
-      dot = warp_sum(dot);
-      if (lane == 0) {
-        tok[3 * DP + kScanCols] = dot;
-        if (MODE == kDelta) tok[3 * DP + kScanCols + 1] = a.beta[t * a.H + h];
-      }
-    }
-  };
-  auto store_chunk = [&](int ch) {
-    const float* ob = outb + (ch & 1) * kScanTok * kScanCols;
-    const int cnt = min(kScanTok, n_tok - ch * kScanTok);
-    for (int i = warp - kScanWarps; i < cnt; i += kLoadWarps) {
-      const size_t t = (size_t)t_begin + ch * kScanTok + i;
-      if (col0 + lane < a.dv) a.o[(t * a.H + h) * a.dv + col0 + lane] = ob[i * kScanCols + lane];
-    }
-  };
+  // the copies never write past d and dv: what lies behind must read as zero
+  for (int i = threadIdx.x; i < scan_smem_bytes<T, NI>() / 4; i += kScanThreads) sm[i] = 0.f;
 
-  float S[4 * NI];
+  f32x2 S[2 * NI];
 #pragma unroll
-  for (int i = 0; i < 4 * NI; ++i) S[i] = 0.f;
+  for (int i = 0; i < 2 * NI; ++i) S[i] = 0ull;
   float* srow = nullptr;
   if (a.state != nullptr && live) {
     srow = a.state + (((size_t)a.slots[s] * a.H + h) * a.dv + col) * DP + r * 4;
     if (a.pos0[s] > 0) {
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        const float4 x = *reinterpret_cast<const float4*>(srow + i * 32);
-        S[4 * i] = x.x; S[4 * i + 1] = x.y; S[4 * i + 2] = x.z; S[4 * i + 3] = x.w;
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(srow + i * 32);
+        S[2 * i] = x.x;
+        S[2 * i + 1] = x.y;
       }
     }
   }
-  if (loader) load_chunk(0);
+  __syncthreads();
+
+  auto issue = [&](int ch) {                           // start the copies of a chunk (this warp's tokens)
+    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+      const size_t t = (size_t)t_begin + ch * kScanTok + i;
+      const T* qp = reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
+      const T* kp = reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
+      const T* vp = reinterpret_cast<const T*>(a.v) + t * a.ldv + (size_t)h * a.dv + col0;
+      const int nv = min(kScanCols, a.dv - col0);
+      float *gd, *bd;
+      T *qd, *kd, *vd;
+      if (kF32) {
+        float* tok = sm + ((ch % kScanRing) * kScanTok + i) * TF;
+        qd = reinterpret_cast<T*>(tok), kd = qd + DP, gd = tok + 2 * DP, vd = reinterpret_cast<T*>(tok + 3 * DP);
+        bd = tok + 3 * DP + kScanCols + 1;
+      } else {
+        uint8_t* rec = raw + ((ch % kScanRing) * kScanTok + i) * R::kRawBytes;
+        gd = reinterpret_cast<float*>(rec), bd = gd + DP, qd = reinterpret_cast<T*>(gd + DP + 4), kd = qd + DP, vd = kd + DP;
+      }
+      warp_copy<T>(qd, qp, a.d, vec, lane);
+      warp_copy<T>(kd, kp, a.d, vec, lane);
+      warp_copy<float>(gd, a.g + (t * a.H + h) * a.d, a.d, vec, lane);
+      warp_copy<T>(vd, vp, nv, vec, lane);
+      if (MODE == kDelta && lane == 0) cp_async4(bd, a.beta + t * a.H + h);
+    }
+    cp_async_commit();
+  };
+  auto prepare = [&](int ch) {                         // a landed chunk: scalars, and fp32 records of bf16 operands
+    cp_async_wait<kScanRing - 2>();
+    __syncwarp();
+    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+      const size_t t = (size_t)t_begin + ch * kScanTok + i;
+      float* tok = sm + ((ch % kBufs) * kScanTok + i) * TF;
+      float dot = 0.f;
+      if (kF32) {
+#pragma unroll
+        for (int c = 0; c < NI; ++c) {
+          const int x = c * 32 + lane;
+          const float p = tok[x] * tok[DP + x];
+          dot += MODE == kWkv ? (x < a.d ? p * a.u[(size_t)h * a.d + x] : 0.f) : p;
+        }
+      } else {
+        const uint8_t* rec = raw + ((ch % kScanRing) * kScanTok + i) * R::kRawBytes;
+        const float* gs = reinterpret_cast<const float*>(rec);
+        const T* qs = vec ? reinterpret_cast<const T*>(gs + DP + 4)
+                          : reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
+        const T* ks = vec ? reinterpret_cast<const T*>(gs + DP + 4) + DP
+                          : reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
+        const T* vs = vec ? reinterpret_cast<const T*>(gs + DP + 4) + 2 * DP
+                          : reinterpret_cast<const T*>(a.v) + t * a.ldv + (size_t)h * a.dv + col0;
+#pragma unroll
+        for (int c = 0; c < NI; ++c) {
+          const int x = c * 32 + lane;
+          const bool in = x < a.d;
+          const float q = in ? to_f<T>(qs[x]) : 0.f, k = in ? to_f<T>(ks[x]) : 0.f;
+          tok[x] = q;
+          tok[DP + x] = k;
+          tok[2 * DP + x] = gs[x];
+          dot += MODE == kWkv ? (in ? q * k * a.u[(size_t)h * a.d + x] : 0.f) : q * k;
+        }
+        tok[3 * DP + lane] = col0 + lane < a.dv ? to_f<T>(vs[lane]) : 0.f;
+        if (lane == 0) tok[3 * DP + kScanCols + 1] = gs[DP];
+      }
+      dot = warp_sum(dot);
+      if (lane == 0) tok[3 * DP + kScanCols] = dot;
+    }
+  };
+  auto store = [&](int ch) {
+    const float* ob = outb + (ch & 1) * kScanTok * kScanCols;
+    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+      const size_t t = (size_t)t_begin + ch * kScanTok + i;
+      if (col0 + lane < a.dv) a.o[(t * a.H + h) * a.dv + col0 + lane] = ob[i * kScanCols + lane];
+    }
+  };
+
+  if (loader) {
+#pragma unroll
+    for (int c = 0; c < kScanRing - 1; ++c) issue(c);
+    prepare(0);
+  }
   __syncthreads();
   for (int ch = 0; ch < n_chunk; ++ch) {
     if (loader) {
-      if (ch + 1 < n_chunk) load_chunk(ch + 1);
-      if (ch > 0) store_chunk(ch - 1);
+      issue(ch + kScanRing - 1);
+      prepare(ch + 1);
+      if (ch > 0) store(ch - 1);
     } else {
-      const float* st = stage[ch & 1];
-      float* ob = outb + (ch & 1) * kScanTok * kScanCols;
+      const float* st = sm + (ch % kBufs) * kScanTok * TF;
       const int cnt = min(kScanTok, n_tok - ch * kScanTok);
-      for (int i = 0; i < cnt; ++i) {
-        const float* tok = st + i * kTokFloats;
+      float out = 0.f;                                 // lane r of a column keeps the output of token r
+      auto token = [&](int i) {
+        const float* tok = st + i * TF;
         const float v = tok[3 * DP + cl], sc = tok[3 * DP + kScanCols];
         if (MODE == kWkv) {
-          float o0 = 0.f, o1 = 0.f;
+          const f32x2 vv = pack2(v, v);
+          f32x2 o0 = 0ull, o1 = 0ull;
 #pragma unroll
           for (int j = 0; j < NI; ++j) {
-            const float4 q = *reinterpret_cast<const float4*>(tok + j * 32 + r * 4);
-            const float4 k = *reinterpret_cast<const float4*>(tok + DP + j * 32 + r * 4);
-            const float4 g = *reinterpret_cast<const float4*>(tok + 2 * DP + j * 32 + r * 4);
-            float* x = S + 4 * j;
-            o0 = fmaf(q.x, x[0], o0); o1 = fmaf(q.y, x[1], o1);
-            o0 = fmaf(q.z, x[2], o0); o1 = fmaf(q.w, x[3], o1);
-            x[0] = fmaf(g.x, x[0], k.x * v); x[1] = fmaf(g.y, x[1], k.y * v);
-            x[2] = fmaf(g.z, x[2], k.z * v); x[3] = fmaf(g.w, x[3], k.w * v);
+            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(tok + j * 32 + r * 4);
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(tok + DP + j * 32 + r * 4);
+            const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 32 + r * 4);
+            o0 = fma2(q.x, S[2 * j], o0);
+            o1 = fma2(q.y, S[2 * j + 1], o1);
+            S[2 * j] = fma2(g.x, S[2 * j], mul2(k.x, vv));
+            S[2 * j + 1] = fma2(g.y, S[2 * j + 1], mul2(k.y, vv));
           }
-          float o = o0 + o1;
+          float o = sum2(o0) + sum2(o1);
           o += __shfl_xor_sync(0xffffffffu, o, 1);
           o += __shfl_xor_sync(0xffffffffu, o, 2);
           o += __shfl_xor_sync(0xffffffffu, o, 4);
-          if (r == 0) ob[i * kScanCols + cl] = fmaf(sc, v, o);
+          if (r == i) out = fmaf(sc, v, o);
         } else {
           const float beta = tok[3 * DP + kScanCols + 1];
-          float k0 = 0.f, k1 = 0.f, q0 = 0.f, q1 = 0.f;
-          float kk[4 * NI];
+          f32x2 k0 = 0ull, k1 = 0ull, q0 = 0ull, q1 = 0ull;
+          f32x2 kk[2 * NI];
 #pragma unroll
           for (int j = 0; j < NI; ++j) {
-            const float4 q = *reinterpret_cast<const float4*>(tok + j * 32 + r * 4);
-            const float4 k = *reinterpret_cast<const float4*>(tok + DP + j * 32 + r * 4);
-            const float4 g = *reinterpret_cast<const float4*>(tok + 2 * DP + j * 32 + r * 4);
-            float* x = S + 4 * j;
-            kk[4 * j] = k.x; kk[4 * j + 1] = k.y; kk[4 * j + 2] = k.z; kk[4 * j + 3] = k.w;
-            x[0] *= g.x; x[1] *= g.y; x[2] *= g.z; x[3] *= g.w;
-            k0 = fmaf(k.x, x[0], k0); k1 = fmaf(k.y, x[1], k1);
-            q0 = fmaf(q.x, x[0], q0); q1 = fmaf(q.y, x[1], q1);
-            k0 = fmaf(k.z, x[2], k0); k1 = fmaf(k.w, x[3], k1);
-            q0 = fmaf(q.z, x[2], q0); q1 = fmaf(q.w, x[3], q1);
+            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(tok + j * 32 + r * 4);
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(tok + DP + j * 32 + r * 4);
+            const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 32 + r * 4);
+            kk[2 * j] = k.x;
+            kk[2 * j + 1] = k.y;
+            S[2 * j] = mul2(S[2 * j], g.x);
+            S[2 * j + 1] = mul2(S[2 * j + 1], g.y);
+            k0 = fma2(k.x, S[2 * j], k0);
+            k1 = fma2(k.y, S[2 * j + 1], k1);
+            q0 = fma2(q.x, S[2 * j], q0);
+            q1 = fma2(q.y, S[2 * j + 1], q1);
           }
           // even lanes reduce the k sum, odd lanes the q sum
-          const float ks = k0 + k1, qs = q0 + q1;
+          const float ks = sum2(k0) + sum2(k1), qs = sum2(q0) + sum2(q1);
           float mine = (r & 1) ? qs : ks;
           mine += __shfl_xor_sync(0xffffffffu, (r & 1) ? ks : qs, 1);
           mine += __shfl_xor_sync(0xffffffffu, mine, 2);
           mine += __shfl_xor_sync(0xffffffffu, mine, 4);
           const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
           const float e = beta * (v - ((r & 1) ? other : mine));
-          if (r == 0) ob[i * kScanCols + cl] = fmaf(sc, e, other);
+          if (r == i) out = fmaf(sc, e, (r & 1) ? mine : other);
+          const f32x2 ee = pack2(e, e);
 #pragma unroll
-          for (int j = 0; j < 4 * NI; ++j) S[j] = fmaf(kk[j], e, S[j]);
+          for (int j = 0; j < 2 * NI; ++j) S[j] = fma2(kk[j], ee, S[j]);
         }
+      };
+      if (cnt == kScanTok) {
+#pragma unroll
+        for (int i = 0; i < kScanTok; ++i) token(i);
+      } else {
+        for (int i = 0; i < cnt; ++i) token(i);
       }
+      outb[(ch & 1) * kScanTok * kScanCols + r * kScanCols + cl] = out;
     }
     __syncthreads();
   }
   if (loader) {
-    store_chunk(n_chunk - 1);
+    store(n_chunk - 1);
   } else if (srow != nullptr) {
 #pragma unroll
-    for (int i = 0; i < NI; ++i)
-      *reinterpret_cast<float4*>(srow + i * 32) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+    for (int i = 0; i < NI; ++i) *reinterpret_cast<ulonglong2*>(srow + i * 32) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
   }
 }
 
 template <int MODE, typename T, int NI>
 int launch_scan(const ScanArgs& a, int n_seq, int vec, cudaStream_t stream) {
-  constexpr int bytes = (2 * kScanTok * (3 * NI * 32 + kScanCols + 4) + 2 * kScanTok * kScanCols) * 4;
+  constexpr int bytes = scan_smem_bytes<T, NI>();
   auto kern = scan_kernel<MODE, T, NI>;
   static bool configured = false;
   if (!configured) {
@@ -214,8 +301,10 @@ int launch_scan(const ScanArgs& a, int n_seq, int vec, cudaStream_t stream) {
 
 template <int MODE, typename T>
 int dispatch_scan(const ScanArgs& a, int n_seq, cudaStream_t stream) {
-  const int v = a.d % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && aligned_to(a.q, 16) && aligned_to(a.k, 16) &&
-                aligned_to(a.g, 16) && aligned_to(a.u, 16);
+  // 16-byte copies: every head starts on a 16-byte boundary and is a multiple of 16 bytes long
+  constexpr int per = 16 / sizeof(T);
+  const int v = a.d % per == 0 && a.dv % per == 0 && a.d % 4 == 0 && a.ldq % per == 0 && a.ldk % per == 0 &&
+                a.ldv % per == 0 && aligned_to(a.q, 16) && aligned_to(a.k, 16) && aligned_to(a.v, 16) && aligned_to(a.g, 16);
   switch ((a.d + 31) / 32) {
     case 1: return launch_scan<MODE, T, 1>(a, n_seq, v, stream);
     case 2: return launch_scan<MODE, T, 2>(a, n_seq, v, stream);
@@ -246,10 +335,27 @@ struct DeltaInArgs {
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+// Sums over the 32 lanes of 16 values per lane: lane l returns the total of value l >> 1.
+__device__ __forceinline__ float warp_sum16(float* v) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 16, n = 8; o >= 2; o >>= 1, n >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i < n) {
+        const float keep = up ? v[i + n] : v[i], give = up ? v[i] : v[i + n];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+      }
+    }
+  }
+  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+}
+
 // blockIdx.x: a q head, a k head, a v head, or the decays of a head; blockIdx.y: chunk of tokens; blockIdx.z: sequence.
 // Thread c is channel c of the head.  Only chunk 0 reaches in front of the sequence, so it alone reads the tail, and
-// it replaces it by the sequence's last inputs afterwards (each thread its own channel).
-template <typename T>
+// it replaces it by the sequence's last inputs afterwards (each thread its own channel).  NT: taps (0: any number).
+template <typename T, int NT>
 __global__ void delta_inputs_kernel(const DeltaInArgs p) {
   __shared__ float red[kConvTok][33];
   const int s = blockIdx.z, sa = p.cu[s], sb = p.cu[s + 1];
@@ -260,18 +366,23 @@ __global__ void delta_inputs_kernel(const DeltaInArgs p) {
   if (head >= 2 * p.G + p.H) {
     head -= 2 * p.G + p.H;
     const float rate = expf(p.A_log[head]);
-    for (int t = t0; t < t1; ++t) {
-      if (c < p.d) {
-        float* z = p.a + (size_t)t * p.H * p.d + head * p.d + c;
-        *z = expf(-rate * softplus_f(*z + p.dt_bias[head * p.d + c]));
-      }
-      if (c == 0) p.beta[(size_t)t * p.H + head] = sigmoid_f(p.b[(size_t)t * p.ldb + head]);
+    float z[kConvTok];
+    if (c < p.d) {
+      float* base = p.a + head * p.d + c;
+#pragma unroll
+      for (int i = 0; i < kConvTok; ++i) z[i] = base[(size_t)min(t0 + i, t1 - 1) * p.H * p.d];
+      const float dt = p.dt_bias[head * p.d + c];
+#pragma unroll
+      for (int i = 0; i < kConvTok; ++i)
+        if (t0 + i < t1) base[(size_t)(t0 + i) * p.H * p.d] = expf(-rate * softplus_f(z[i] + dt));
     }
+    if (c < t1 - t0) p.beta[(size_t)(t0 + c) * p.H + head] = sigmoid_f(p.b[(size_t)(t0 + c) * p.ldb + head]);
     return;
   }
   const bool is_v = head >= 2 * p.G;
   const int width = is_v ? p.dv : p.d;
-  const int C = 2 * p.G * p.d + p.H * p.dv, n1 = p.n_taps - 1;
+  const int n_taps = NT > 0 ? NT : p.n_taps;
+  const int C = 2 * p.G * p.d + p.H * p.dv, n1 = n_taps - 1;
   const int ch = is_v ? 2 * p.G * p.d + (head - 2 * p.G) * p.dv + c : head * p.d + c;
   const T* x = reinterpret_cast<const T*>(p.x) + ch;
   float y[kConvTok];
@@ -280,15 +391,21 @@ __global__ void delta_inputs_kernel(const DeltaInArgs p) {
   if (c < width) {
     T* tail = p.tail != nullptr ? reinterpret_cast<T*>(p.tail) + ((size_t)p.slots[s] * C + ch) * n1 : nullptr;
     const bool past = tail != nullptr && p.pos0[s] > 0;
-    for (int j = 0; j <= n1; ++j) {                       // tap of the input j tokens back
-      const float w = p.taps[(size_t)ch * p.n_taps + n1 - j];
+    constexpr int kReach = NT > 0 ? NT - 1 : kConvTok;
+    float w[kReach + kConvTok];                           // inputs t0 - kReach .. t0 + 15
 #pragma unroll
-      for (int i = 0; i < kConvTok; ++i) {
-        const int t = t0 + i - j;
-        if (t0 + i < t1) {
-          if (t >= sa) y[i] = fmaf(w, to_f<T>(x[(size_t)t * p.ldx]), y[i]);
-          else if (past) y[i] = fmaf(w, to_f<T>(tail[n1 + t - sa]), y[i]);
-        }
+    for (int i = 0; i < kReach + kConvTok; ++i) {
+      const int t = t0 - kReach + i;
+      w[i] = 0.f;
+      if (t >= sa) w[i] = to_f<T>(x[(size_t)min(t, t1 - 1) * p.ldx]);
+      else if (past && t >= sa - n1) w[i] = to_f<T>(tail[n1 + t - sa]);
+    }
+#pragma unroll
+    for (int j = 0; j <= kReach; ++j) {                   // tap of the input j tokens back
+      if (j <= n1) {
+        const float tap = p.taps[(size_t)ch * n_taps + n1 - j];
+#pragma unroll
+        for (int i = 0; i < kConvTok; ++i) y[i] = fmaf(tap, w[kReach + i - j], y[i]);
       }
     }
 #pragma unroll
@@ -302,26 +419,42 @@ __global__ void delta_inputs_kernel(const DeltaInArgs p) {
     }
   }
   if (is_v) {
-    if (c < width)
-      for (int i = 0; t0 + i < t1; ++i) p.v[((size_t)(t0 + i) * p.H + head - 2 * p.G) * p.dv + c] = y[i];
+    if (c < width) {
+      float* out = p.v + (size_t)(head - 2 * p.G) * p.dv + c;
+#pragma unroll
+      for (int i = 0; i < kConvTok; ++i)
+        if (t0 + i < t1) out[(size_t)(t0 + i) * p.H * p.dv] = y[i];
+    }
     return;
   }
+  float sq[kConvTok];
 #pragma unroll
-  for (int i = 0; i < kConvTok; ++i) {
-    const float ss = warp_sum(y[i] * y[i]);
-    if (lane == 0) red[i][warp] = ss;
-  }
+  for (int i = 0; i < kConvTok; ++i) sq[i] = y[i] * y[i];
+  const float ss = warp_sum16(sq);
+  if (!(lane & 1)) red[lane >> 1][warp] = ss;
   __syncthreads();
   const bool is_q = head < p.G;
   float* out = (is_q ? p.q : p.k) + (size_t)(is_q ? head : head - p.G) * p.d + c;
   const float mul = is_q ? 1.f / sqrtf((float)p.d) : 1.f;
+  if (threadIdx.x < kConvTok) {
+    float t = 0.f;
+    for (int w = 0; w < nw; ++w) t += red[threadIdx.x][w];
+    red[threadIdx.x][32] = mul / sqrtf(t + 1e-6f);
+  }
+  __syncthreads();
 #pragma unroll
-  for (int i = 0; i < kConvTok; ++i) {
-    if (t0 + i < t1 && c < width) {
-      float ss = 0.f;
-      for (int w = 0; w < nw; ++w) ss += red[i][w];
-      out[(size_t)(t0 + i) * p.G * p.d] = y[i] / sqrtf(ss + 1e-6f) * mul;
-    }
+  for (int i = 0; i < kConvTok; ++i)
+    if (t0 + i < t1 && c < width) out[(size_t)(t0 + i) * p.G * p.d] = y[i] * red[i][32];
+}
+
+template <typename T>
+static void launch_delta_inputs(const DeltaInArgs& p, dim3 grid, int threads, cudaStream_t stream) {
+  switch (p.n_taps) {
+    case 1: delta_inputs_kernel<T, 1><<<grid, threads, 0, stream>>>(p); break;
+    case 2: delta_inputs_kernel<T, 2><<<grid, threads, 0, stream>>>(p); break;
+    case 3: delta_inputs_kernel<T, 3><<<grid, threads, 0, stream>>>(p); break;
+    case 4: delta_inputs_kernel<T, 4><<<grid, threads, 0, stream>>>(p); break;
+    default: delta_inputs_kernel<T, 0><<<grid, threads, 0, stream>>>(p);
   }
 }
 
@@ -359,7 +492,7 @@ ELL_API int ell_delta_inputs(const void* x, const float* taps, float* a, const f
   DeltaInArgs p{x, taps, a, A_log, dt_bias, b, q, k, v, beta, tail, cu, slots, pos0, H, G, d, dv, n_taps, ldx, ldb};
   dim3 grid(2 * G + 2 * H, chunks, n_seq);
   const int threads = (width + 31) / 32 * 32;
-  if (is_bf16) delta_inputs_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(p);
-  else delta_inputs_kernel<float><<<grid, threads, 0, stream>>>(p);
+  if (is_bf16) launch_delta_inputs<__nv_bfloat16>(p, grid, threads, stream);
+  else launch_delta_inputs<float>(p, grid, threads, stream);
   return launch_status();
 }

@@ -73,11 +73,24 @@ __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float* f) {
   }
 }
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// Accurate expf, and a division of at most 2 ulp (0 for a denominator above 2^126, which is the limit here).
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.f + expf(-z)); }
+// 0.5 (1 + tanh(x)) = sigmoid(2 x)
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return __fdividef(z, 1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
+
+// Asynchronous copies into shared memory (16-byte aligned, 16 bytes; or 4 and 4).
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 inline bool aligned_to(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
 
