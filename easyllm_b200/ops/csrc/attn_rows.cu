@@ -12,7 +12,7 @@
 
 namespace ell {
 
-constexpr int kArThreads = 128, kArRep = 8;
+constexpr int kArThreads = 128, kArRep = 8;   // kArRep: most query heads of a CTA (REP: 4 or 8)
 
 struct AttnRowsArgs {
   const void *q, *k, *v;
@@ -29,7 +29,7 @@ struct ArLayout {
   int dp, krow, vrow, kgroups;    // padded key size; row strides in elements; key shares of the weighted sum
   int stage, bytes;               // elements of a stage; total bytes
 };
-__host__ __device__ inline ArLayout ar_layout(int d, int dv, int esz, int KT) {
+__host__ __device__ inline ArLayout ar_layout(int d, int dv, int esz, int KT, int REP) {
   ArLayout l;
   l.dp = (d + 63) / 64 * 64;
   l.krow = l.dp + 16 / esz;
@@ -38,24 +38,24 @@ __host__ __device__ inline ArLayout ar_layout(int d, int dv, int esz, int KT) {
   l.kgroups = 1;
   while (2 * l.kgroups * oct <= kArThreads && 2 * l.kgroups <= KT / 4 && l.kgroups < 16) l.kgroups *= 2;
   l.stage = KT * (l.krow + l.vrow);
-  const int head = (kArRep * l.dp + kArRep * KT + kArRep * 4) * 4;
-  const int a = 2 * l.stage * esz, b = l.kgroups * kArRep * oct * 8 * 4;   // the sums reuse the stages
+  const int head = (REP * l.dp + REP * KT + REP * 4) * 4;
+  const int a = 2 * l.stage * esz, b = l.kgroups * REP * oct * 8 * 4;   // the sums reuse the stages
   l.bytes = head + (a > b ? a : b);
   return l;
 }
 
-template <typename T, int KT, bool VEC>
+template <typename T, int KT, int REP, bool VEC>
 __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArgs a) {
   extern __shared__ __align__(16) float sm[];
-  const ArLayout L = ar_layout(a.d, a.dv, sizeof(T), KT);
-  const int t = blockIdx.x, rep = a.H / a.G, groups = (rep + kArRep - 1) / kArRep;
-  const int g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * kArRep;
-  const int nh = min(kArRep, g * rep + rep - h0);
+  const ArLayout L = ar_layout(a.d, a.dv, sizeof(T), KT, REP);
+  const int t = blockIdx.x, rep = a.H / a.G, groups = (rep + REP - 1) / REP;
+  const int g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * REP;
+  const int nh = min(REP, g * rep + rep - h0);
   const int split = blockIdx.z, dp = L.dp, oct = (a.dv + 7) / 8;
   float* qs = sm;
-  float* p = qs + kArRep * dp;
-  float* stat = p + kArRep * KT;                    // max, sum, rescale
-  T* stages = reinterpret_cast<T*>(stat + kArRep * 4);
+  float* p = qs + REP * dp;
+  float* stat = p + REP * KT;                    // max, sum, rescale
+  T* stages = reinterpret_cast<T*>(stat + REP * 4);
   const int len = a.len[t];
   const size_t base = a.base[t];
   const int k0 = split * a.range, k1 = min(k0 + a.range, len);
@@ -63,12 +63,12 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
   // rows and columns the copies leave out must read as zero
   for (int i = threadIdx.x; i < 2 * L.stage * (int)sizeof(T) / 16; i += kArThreads)
     reinterpret_cast<uint4*>(stages)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = threadIdx.x; i < kArRep * dp; i += kArThreads) {
+  for (int i = threadIdx.x; i < REP * dp; i += kArThreads) {
     const int h = i / dp, c = i % dp;
     qs[i] = h < nh && c < a.d
                 ? to_f<T>(reinterpret_cast<const T*>(a.q)[(size_t)t * a.ldq + (size_t)(h0 + h) * a.d + c]) * a.scale : 0.f;
   }
-  if (threadIdx.x < kArRep) {
+  if (threadIdx.x < REP) {
     stat[threadIdx.x * 4] = -INFINITY;
     stat[threadIdx.x * 4 + 1] = 0.f;
   }
@@ -101,9 +101,9 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
   // weighted sum: this thread's eight columns and its share of a tile's keys
   const int my_oct = threadIdx.x % oct, my_share = threadIdx.x / oct, share = KT / L.kgroups;
   const bool adds = my_share < L.kgroups;
-  float acc[kArRep][8];
+  float acc[REP][8];
 #pragma unroll
-  for (int h = 0; h < kArRep; ++h)
+  for (int h = 0; h < REP; ++h)
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[h][j] = 0.f;
   const int l8 = lane & 7, grp = warp * 4 + (lane >> 3);          // 16 groups of 8 lanes
@@ -121,9 +121,9 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
     const T* ks = stages + buf * L.stage;
     const T* vs = ks + KT * L.krow;
     // scores: a group takes keys grp, grp + 16, ...
-    float sc[kArRep][KJ];
+    float sc[REP][KJ];
 #pragma unroll
-    for (int h = 0; h < kArRep; ++h)
+    for (int h = 0; h < REP; ++h)
 #pragma unroll
       for (int j = 0; j < KJ; ++j) sc[h][j] = 0.f;
     for (int c = l8 * 8; c < dp; c += 64) {
@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
 #pragma unroll
       for (int j = 0; j < KJ; ++j) load_v<8>(ks + (grp + 16 * j) * L.krow + c, kv[j]);
 #pragma unroll
-      for (int h = 0; h < kArRep; ++h) {
+      for (int h = 0; h < REP; ++h) {
         if (h < nh) {
           const float4 q0 = *reinterpret_cast<const float4*>(qs + h * dp + c);
           const float4 q1 = *reinterpret_cast<const float4*>(qs + h * dp + c + 4);
@@ -146,7 +146,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
       }
     }
 #pragma unroll
-    for (int h = 0; h < kArRep; ++h) {
+    for (int h = 0; h < REP; ++h) {
       if (h < nh) {
 #pragma unroll
         for (int j = 0; j < KJ; ++j) {
@@ -189,7 +189,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
     __syncthreads();
     if (adds) {
 #pragma unroll
-      for (int h = 0; h < kArRep; ++h) {
+      for (int h = 0; h < REP; ++h) {
         if (h < nh) {
           const float al = stat[h * 4 + 2];
           if (al != 1.f) {
@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
 #pragma unroll
         for (int x = 0; x < 4; ++x) load_v<8>(vp + (i + x) * L.vrow, vv[x]);
 #pragma unroll
-        for (int h = 0; h < kArRep; ++h) {
+        for (int h = 0; h < REP; ++h) {
           if (h < nh) {
             const float4 w = *reinterpret_cast<const float4*>(p + h * KT + my_share * share + i);
 #pragma unroll
@@ -220,14 +220,14 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
   float* sums = reinterpret_cast<float*>(stages);
   if (adds) {
 #pragma unroll
-    for (int h = 0; h < kArRep; ++h)
-      if (h < nh) store_v<8>(sums + ((my_share * kArRep + h) * oct + my_oct) * 8, acc[h]);
+    for (int h = 0; h < REP; ++h)
+      if (h < nh) store_v<8>(sums + ((my_share * REP + h) * oct + my_oct) * 8, acc[h]);
   }
   __syncthreads();
   for (int i = threadIdx.x; i < nh * a.dv; i += kArThreads) {
     const int h = i / a.dv, c = i % a.dv;
     float o = 0.f;
-    for (int x = 0; x < L.kgroups; ++x) o += sums[(x * kArRep + h) * oct * 8 + c];
+    for (int x = 0; x < L.kgroups; ++x) o += sums[(x * REP + h) * oct * 8 + c];
     const float m = stat[h * 4], l = stat[h * 4 + 1];
     if (a.splits == 1) {
       float den = l, f = 1.f;
@@ -265,10 +265,13 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_merge_kernel(const AttnR
   }
 }
 
+// Query heads a CTA takes.
+static int ar_rep(int rep) { return rep <= 4 ? 4 : kArRep; }
+
 // Ranges per row: enough CTAs to fill the GPU a few times, about 256 keys each at least.
 static int attn_rows_splits(int n, int H, int G, int max_len) {
   const int rep = H / G;
-  const long long ctas = (long long)n * G * ((rep + kArRep - 1) / kArRep);
+  const long long ctas = (long long)n * G * ((rep + ar_rep(rep) - 1) / ar_rep(rep));
   long long s = (4LL * kNumSMs + ctas - 1) / ctas;
   const long long most = (max_len + 255) / 256;
   if (s > most) s = most;
@@ -276,10 +279,10 @@ static int attn_rows_splits(int n, int H, int G, int max_len) {
   return s < 1 ? 1 : (int)s;
 }
 
-template <typename T, int KT, bool VEC>
+template <typename T, int KT, int REP, bool VEC>
 static int launch_attn_rows_kt(const AttnRowsArgs& a, dim3 grid, cudaStream_t stream) {
-  const int bytes = ar_layout(a.d, a.dv, sizeof(T), KT).bytes;
-  auto kern = attn_rows_kernel<T, KT, VEC>;
+  const int bytes = ar_layout(a.d, a.dv, sizeof(T), KT, REP).bytes;
+  auto kern = attn_rows_kernel<T, KT, REP, VEC>;
   static int configured = 0;
   if (bytes > configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
@@ -291,11 +294,11 @@ static int launch_attn_rows_kt(const AttnRowsArgs& a, dim3 grid, cudaStream_t st
   return launch_status();
 }
 
-template <typename T>
+template <typename T, int REP>
 static int launch_attn_rows(const AttnRowsArgs& a, dim3 grid, bool vec, cudaStream_t stream) {
-  const bool small = ar_layout(a.d, a.dv, sizeof(T), 64).bytes > 160 * 1024;      // very wide fp32 heads: short tiles
-  if (small) return vec ? launch_attn_rows_kt<T, 16, true>(a, grid, stream) : launch_attn_rows_kt<T, 16, false>(a, grid, stream);
-  return vec ? launch_attn_rows_kt<T, 64, true>(a, grid, stream) : launch_attn_rows_kt<T, 64, false>(a, grid, stream);
+  const bool small = ar_layout(a.d, a.dv, sizeof(T), 32, REP).bytes > 160 * 1024;      // very wide fp32 heads: short tiles
+  if (small) return vec ? launch_attn_rows_kt<T, 16, REP, true>(a, grid, stream) : launch_attn_rows_kt<T, 16, REP, false>(a, grid, stream);
+  return vec ? launch_attn_rows_kt<T, 32, REP, true>(a, grid, stream) : launch_attn_rows_kt<T, 32, REP, false>(a, grid, stream);
 }
 
 }  // namespace ell
@@ -318,10 +321,12 @@ ELL_API int ell_attn_rows(const void* q, const void* k, const void* v, void* out
   a.splits = attn_rows_splits(n, H, G, max_len);
   a.range = ((max_len + a.splits - 1) / a.splits + 63) / 64 * 64;
   if (a.splits > 1 && part == nullptr) return -2;
-  const int rep = H / G;
-  dim3 grid(n, G * ((rep + kArRep - 1) / kArRep), a.splits);
+  const int rep = H / G, per = ar_rep(rep);
+  dim3 grid(n, G * ((rep + per - 1) / per), a.splits);
   const int esz = is_bf16 ? 2 : 4;
   const bool vec = (d * esz) % 16 == 0 && (dv * esz) % 16 == 0 && (ldk * esz) % 16 == 0 && (ldv * esz) % 16 == 0 &&
                    aligned_to(k, 16) && aligned_to(v, 16);
-  return is_bf16 ? launch_attn_rows<__nv_bfloat16>(a, grid, vec, stream) : launch_attn_rows<float>(a, grid, vec, stream);
+  if (is_bf16)
+    return per == 4 ? launch_attn_rows<__nv_bfloat16, 4>(a, grid, vec, stream) : launch_attn_rows<__nv_bfloat16, 8>(a, grid, vec, stream);
+  return per == 4 ? launch_attn_rows<float, 4>(a, grid, vec, stream) : launch_attn_rows<float, 8>(a, grid, vec, stream);
 }

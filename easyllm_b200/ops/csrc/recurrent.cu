@@ -5,22 +5,23 @@
 // A state matrix S [d key rows x dv value columns] of one head evolves column by column without mixing columns:
 //   time mixing   o_j = sum_i r_i (S_ij + u_i k_i v_j),          S_ij <- w_i S_ij + k_i v_j
 //   delta rule    S_ij <- g_i S_ij,  e_j = beta (v_j - sum_i k_i S_ij),  S_ij <- S_ij + k_i e_j,  o_j = sum_i q_i S_ij
-// so a CTA owns 32 columns of one (sequence, head) and no CTA waits for another.  Eight lanes share a column: lane r
-// keeps rows 32 i + 4 r .. + 3 in registers for the whole sequence.  Both sums of the delta rule are taken from the
-// decayed state at once (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the
-// token-to-token chain.
-// Warps 0-7 run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Warps 8-11 copy the operands of the coming tokens
-// into a ring of shared-memory stages with cp.async (three stages ahead), convert bf16 operands to fp32, compute the
-// per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous tokens' outputs.
+// so a CTA owns 32 columns of one (sequence, head) and no CTA waits for another.  A thread keeps 4 columns x 4 or 8 key
+// rows in registers for the whole sequence (8 to 32 lanes share the columns): every operand word read from shared memory
+// then serves four columns, which matters because filling registers from shared memory, not the arithmetic, is what
+// limits a scan.  Both sums of the delta rule are taken from the decayed state at once
+// (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the token-to-token chain; the sums of
+// the thread's columns are reduced together, halving the number of values with every step.
+// Consumer warps run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Four more warps copy the operands of the coming
+// tokens into a ring of shared-memory stages with cp.async (three stages ahead), convert bf16 operands to fp32, compute
+// the per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous tokens' outputs.
 #include "vec.cuh"
 
 namespace ell {
 
 constexpr int kScanCols = 32;         // value columns of a CTA
-constexpr int kScanTok = 8;           // tokens per stage (one per lane of a column's group: see the outputs)
+constexpr int kScanTok = 8;           // tokens per stage
 constexpr int kScanRing = 4;
-constexpr int kScanWarps = 8, kLoadWarps = 4;
-constexpr int kScanThreads = (kScanWarps + kLoadWarps) * 32;
+constexpr int kLoadWarps = 4;
 
 enum ScanMode { kWkv = 0, kDelta = 1 };
 
@@ -69,25 +70,55 @@ __device__ __forceinline__ void warp_copy(T* dst, const T* src, int n, bool vec,
   }
 }
 
-// Token record the recurrence reads: q | k | g | v | scalar, beta (fp32).  Raw bf16 record: g | beta (fp32), q | k | v.
-template <int NI>
+// Thread layout for heads of up to DP key rows (32, 64, 128 or 256): kLanes lanes hold the rows 4 l + 4 kLanes j .. + 3
+// (j < kJ) of four columns.  Token record the recurrence reads: q | k | g | v | scalar, beta (fp32).  Raw bf16 record:
+// g | beta (fp32), q | k | v.
+template <int DP>
 struct ScanTok {
-  static constexpr int kDp = NI * 32;
-  static constexpr int kFloats = 3 * kDp + kScanCols + 4;
-  static constexpr int kRawBytes = (kDp + 4) * 4 + (2 * kDp + kScanCols) * 2;
+  static constexpr int kLanes = DP <= 64 ? 8 : DP / 8;
+  static constexpr int kJ = DP / (4 * kLanes);
+  static constexpr int kWarpCols = 4 * (32 / kLanes);
+  static constexpr int kWarps = kScanCols / kWarpCols;             // consumer warps
+  static constexpr int kThreads = (kWarps + kLoadWarps) * 32;
+  static constexpr int kFloats = 3 * DP + kScanCols + 4;
+  static constexpr int kRawBytes = (DP + 4) * 4 + (2 * DP + kScanCols) * 2;
 };
-template <typename T, int NI>
+template <typename T, int DP>
 __host__ __device__ constexpr int scan_smem_bytes() {
-  using R = ScanTok<NI>;
+  using R = ScanTok<DP>;
   const int out = 2 * kScanTok * kScanCols * 4;
   return sizeof(T) == 4 ? kScanRing * kScanTok * R::kFloats * 4 + out
                         : 2 * kScanTok * R::kFloats * 4 + kScanRing * kScanTok * R::kRawBytes + out;
 }
 
-template <int MODE, typename T, int NI>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, int vec) {
-  using R = ScanTok<NI>;
-  constexpr int DP = R::kDp, TF = R::kFloats;
+// Sums over the L lanes of a group of NV values per lane.  Each step halves the values a lane keeps (lanes with bit
+// L / 2 set take the upper half, then L / 4, ...) until one is left, which is then summed over the remaining lanes.
+template <int NV, int L>
+__device__ __forceinline__ float reduce_columns(float* v, int l) {
+  int n = NV;
+#pragma unroll
+  for (int o = L / 2; o >= 1; o >>= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool up = l & o;
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i) {
+        if (i < n) {
+          const float keep = up ? v[i + n] : v[i], give = up ? v[i] : v[i + n];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+      }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+  return v[0];
+}
+
+template <int MODE, typename T, int DP>
+__global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanArgs a, int vec) {
+  using R = ScanTok<DP>;
+  constexpr int TF = R::kFloats, L = R::kLanes, J = R::kJ;
   constexpr bool kF32 = sizeof(T) == 4;
   constexpr int kBufs = kF32 ? kScanRing : 2;          // fp32 records: the ring itself, or two converted stages
   extern __shared__ __align__(16) float sm[];
@@ -99,34 +130,40 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
   const int hk = h / (a.H / a.G);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n_chunk = (n_tok + kScanTok - 1) / kScanTok;
-  const bool loader = warp >= kScanWarps;
-  const int r = lane & 7;
-  const int cl = (warp & 7) * 4 + (lane >> 3);         // column within the CTA
-  const int col = col0 + cl;
-  const bool live = !loader && col < a.dv;
+  const bool loader = warp >= R::kWarps;
+  const int lw = warp - R::kWarps;                     // loader warp
+  const int l = lane % L;                              // row slice
+  const int cl = warp * R::kWarpCols + lane / L * 4;   // first of the thread's columns within the CTA
 
   // the copies never write past d and dv: what lies behind must read as zero
-  for (int i = threadIdx.x; i < scan_smem_bytes<T, NI>() / 4; i += kScanThreads) sm[i] = 0.f;
+  for (int i = threadIdx.x; i < scan_smem_bytes<T, DP>() / 16; i += R::kThreads)
+    reinterpret_cast<uint4*>(sm)[i] = make_uint4(0, 0, 0, 0);
 
-  f32x2 S[2 * NI];
+  f32x2 S[4][2 * J];                                   // [column][pair of rows]
 #pragma unroll
-  for (int i = 0; i < 2 * NI; ++i) S[i] = 0ull;
+  for (int c = 0; c < 4; ++c)
+#pragma unroll
+    for (int i = 0; i < 2 * J; ++i) S[c][i] = 0ull;
+  const int sp = (a.d + 31) / 32 * 32;                 // row stride of the stored state
   float* srow = nullptr;
-  if (a.state != nullptr && live) {
-    srow = a.state + (((size_t)a.slots[s] * a.H + h) * a.dv + col) * DP + r * 4;
+  if (a.state != nullptr && !loader) {
+    srow = a.state + (((size_t)a.slots[s] * a.H + h) * a.dv + col0 + cl) * sp + l * 4;
     if (a.pos0[s] > 0) {
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(srow + i * 32);
-        S[2 * i] = x.x;
-        S[2 * i + 1] = x.y;
-      }
+      for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int j = 0; j < J; ++j)
+          if (col0 + cl + c < a.dv && l * 4 + j * 4 * L < sp) {
+            const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(srow + c * sp + j * 4 * L);
+            S[c][2 * j] = x.x;
+            S[c][2 * j + 1] = x.y;
+          }
     }
   }
   __syncthreads();
 
   auto issue = [&](int ch) {                           // start the copies of a chunk (this warp's tokens)
-    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
       const size_t t = (size_t)t_begin + ch * kScanTok + i;
       const T* qp = reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
       const T* kp = reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
@@ -153,13 +190,13 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
   auto prepare = [&](int ch) {                         // a landed chunk: scalars, and fp32 records of bf16 operands
     cp_async_wait<kScanRing - 2>();
     __syncwarp();
-    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
       const size_t t = (size_t)t_begin + ch * kScanTok + i;
       float* tok = sm + ((ch % kBufs) * kScanTok + i) * TF;
       float dot = 0.f;
       if (kF32) {
 #pragma unroll
-        for (int c = 0; c < NI; ++c) {
+        for (int c = 0; c < DP / 32; ++c) {
           const int x = c * 32 + lane;
           const float p = tok[x] * tok[DP + x];
           dot += MODE == kWkv ? (x < a.d ? p * a.u[(size_t)h * a.d + x] : 0.f) : p;
@@ -174,7 +211,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
         const T* vs = vec ? reinterpret_cast<const T*>(gs + DP + 4) + 2 * DP
                           : reinterpret_cast<const T*>(a.v) + t * a.ldv + (size_t)h * a.dv + col0;
 #pragma unroll
-        for (int c = 0; c < NI; ++c) {
+        for (int c = 0; c < DP / 32; ++c) {
           const int x = c * 32 + lane;
           const bool in = x < a.d;
           const float q = in ? to_f<T>(qs[x]) : 0.f, k = in ? to_f<T>(ks[x]) : 0.f;
@@ -192,7 +229,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
   };
   auto store = [&](int ch) {
     const float* ob = outb + (ch & 1) * kScanTok * kScanCols;
-    for (int i = warp - kScanWarps; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
+    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
       const size_t t = (size_t)t_begin + ch * kScanTok + i;
       if (col0 + lane < a.dv) a.o[(t * a.H + h) * a.dv + col0 + lane] = ob[i * kScanCols + lane];
     }
@@ -212,67 +249,86 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
     } else {
       const float* st = sm + (ch % kBufs) * kScanTok * TF;
       const int cnt = min(kScanTok, n_tok - ch * kScanTok);
-      float out = 0.f;                                 // lane r of a column keeps the output of token r
-      auto token = [&](int i) {
+      float* ob = outb + (ch & 1) * kScanTok * kScanCols;
+      // after the reduction a lane holds the sum of one column (and, in the delta rule, of k or of q)
+      constexpr int kC1 = MODE == kDelta ? L / 4 : L / 2, kC0 = kC1 / 2;
+      const int my_c = (l & kC1 ? 2 : 0) + (l & kC0 ? 1 : 0);
+      const bool is_q = MODE == kWkv || (l & (L / 2));
+      const bool writes = is_q && (l & (kC0 - 1)) == 0;
+      float out[kScanTok];
+      auto token = [&](int i) -> float {
         const float* tok = st + i * TF;
-        const float v = tok[3 * DP + cl], sc = tok[3 * DP + kScanCols];
-        if (MODE == kWkv) {
-          const f32x2 vv = pack2(v, v);
-          f32x2 o0 = 0ull, o1 = 0ull;
+        const float sc = tok[3 * DP + kScanCols], v_mine = tok[3 * DP + cl + my_c];
+        ulonglong2 q[J], k[J], g[J];
 #pragma unroll
-          for (int j = 0; j < NI; ++j) {
-            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(tok + j * 32 + r * 4);
-            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(tok + DP + j * 32 + r * 4);
-            const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 32 + r * 4);
-            o0 = fma2(q.x, S[2 * j], o0);
-            o1 = fma2(q.y, S[2 * j + 1], o1);
-            S[2 * j] = fma2(g.x, S[2 * j], mul2(k.x, vv));
-            S[2 * j + 1] = fma2(g.y, S[2 * j + 1], mul2(k.y, vv));
+        for (int j = 0; j < J; ++j) {
+          q[j] = *reinterpret_cast<const ulonglong2*>(tok + j * 4 * L + l * 4);
+          k[j] = *reinterpret_cast<const ulonglong2*>(tok + DP + j * 4 * L + l * 4);
+          g[j] = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 4 * L + l * 4);
+        }
+        if (MODE == kWkv) {
+          const float4 v4 = *reinterpret_cast<const float4*>(tok + 3 * DP + cl);
+          const float v[4] = {v4.x, v4.y, v4.z, v4.w};
+          float sum[4];
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const f32x2 vv = pack2(v[c], v[c]);
+            f32x2 o = 0ull;
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+              o = fma2(q[j].x, S[c][2 * j], o);
+              o = fma2(q[j].y, S[c][2 * j + 1], o);
+              S[c][2 * j] = fma2(g[j].x, S[c][2 * j], mul2(k[j].x, vv));
+              S[c][2 * j + 1] = fma2(g[j].y, S[c][2 * j + 1], mul2(k[j].y, vv));
+            }
+            sum[c] = sum2(o);
           }
-          float o = sum2(o0) + sum2(o1);
-          o += __shfl_xor_sync(0xffffffffu, o, 1);
-          o += __shfl_xor_sync(0xffffffffu, o, 2);
-          o += __shfl_xor_sync(0xffffffffu, o, 4);
-          if (r == i) out = fmaf(sc, v, o);
+          return fmaf(sc, v_mine, reduce_columns<4, L>(sum, l));
         } else {
           const float beta = tok[3 * DP + kScanCols + 1];
-          f32x2 k0 = 0ull, k1 = 0ull, q0 = 0ull, q1 = 0ull;
-          f32x2 kk[2 * NI];
+          float sum[8];
 #pragma unroll
-          for (int j = 0; j < NI; ++j) {
-            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(tok + j * 32 + r * 4);
-            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(tok + DP + j * 32 + r * 4);
-            const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 32 + r * 4);
-            kk[2 * j] = k.x;
-            kk[2 * j + 1] = k.y;
-            S[2 * j] = mul2(S[2 * j], g.x);
-            S[2 * j + 1] = mul2(S[2 * j + 1], g.y);
-            k0 = fma2(k.x, S[2 * j], k0);
-            k1 = fma2(k.y, S[2 * j + 1], k1);
-            q0 = fma2(q.x, S[2 * j], q0);
-            q1 = fma2(q.y, S[2 * j + 1], q1);
+          for (int c = 0; c < 4; ++c) {
+            f32x2 ks = 0ull, qs = 0ull;
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+              S[c][2 * j] = mul2(S[c][2 * j], g[j].x);
+              S[c][2 * j + 1] = mul2(S[c][2 * j + 1], g[j].y);
+              ks = fma2(k[j].x, S[c][2 * j], ks);
+              qs = fma2(q[j].x, S[c][2 * j], qs);
+              ks = fma2(k[j].y, S[c][2 * j + 1], ks);
+              qs = fma2(q[j].y, S[c][2 * j + 1], qs);
+            }
+            sum[c] = sum2(ks);
+            sum[4 + c] = sum2(qs);
           }
-          // even lanes reduce the k sum, odd lanes the q sum
-          const float ks = sum2(k0) + sum2(k1), qs = sum2(q0) + sum2(q1);
-          float mine = (r & 1) ? qs : ks;
-          mine += __shfl_xor_sync(0xffffffffu, (r & 1) ? ks : qs, 1);
-          mine += __shfl_xor_sync(0xffffffffu, mine, 2);
-          mine += __shfl_xor_sync(0xffffffffu, mine, 4);
-          const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
-          const float e = beta * (v - ((r & 1) ? other : mine));
-          if (r == i) out = fmaf(sc, e, (r & 1) ? mine : other);
-          const f32x2 ee = pack2(e, e);
+          const float mine = reduce_columns<8, L>(sum, l);
+          const float e = beta * (v_mine - mine);      // of the lanes that hold a k sum
 #pragma unroll
-          for (int j = 0; j < 2 * NI; ++j) S[j] = fma2(kk[j], ee, S[j]);
+          for (int c = 0; c < 4; ++c) {
+            const float ec = __shfl_sync(0xffffffffu, e, (lane & ~(L - 1)) + (c & 2 ? kC1 : 0) + (c & 1 ? kC0 : 0));
+            const f32x2 ee = pack2(ec, ec);
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+              S[c][2 * j] = fma2(k[j].x, ee, S[c][2 * j]);
+              S[c][2 * j + 1] = fma2(k[j].y, ee, S[c][2 * j + 1]);
+            }
+          }
+          return fmaf(sc, __shfl_xor_sync(0xffffffffu, e, L / 2), mine);
         }
       };
       if (cnt == kScanTok) {
 #pragma unroll
-        for (int i = 0; i < kScanTok; ++i) token(i);
+        for (int i = 0; i < kScanTok; ++i) out[i] = token(i);
+#pragma unroll
+        for (int i = 0; i < kScanTok; ++i)
+          if (writes) ob[i * kScanCols + cl + my_c] = out[i];
       } else {
-        for (int i = 0; i < cnt; ++i) token(i);
+        for (int i = 0; i < cnt; ++i) {
+          const float o = token(i);
+          if (writes) ob[i * kScanCols + cl + my_c] = o;
+        }
       }
-      outb[(ch & 1) * kScanTok * kScanCols + r * kScanCols + cl] = out;
     }
     __syncthreads();
   }
@@ -280,14 +336,18 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const ScanArgs a, in
     store(n_chunk - 1);
   } else if (srow != nullptr) {
 #pragma unroll
-    for (int i = 0; i < NI; ++i) *reinterpret_cast<ulonglong2*>(srow + i * 32) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int j = 0; j < J; ++j)
+        if (col0 + cl + c < a.dv && l * 4 + j * 4 * L < sp)
+          *reinterpret_cast<ulonglong2*>(srow + c * sp + j * 4 * L) = make_ulonglong2(S[c][2 * j], S[c][2 * j + 1]);
   }
 }
 
-template <int MODE, typename T, int NI>
+template <int MODE, typename T, int DP>
 int launch_scan(const ScanArgs& a, int n_seq, int vec, cudaStream_t stream) {
-  constexpr int bytes = scan_smem_bytes<T, NI>();
-  auto kern = scan_kernel<MODE, T, NI>;
+  constexpr int bytes = scan_smem_bytes<T, DP>();
+  auto kern = scan_kernel<MODE, T, DP>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
@@ -295,7 +355,7 @@ int launch_scan(const ScanArgs& a, int n_seq, int vec, cudaStream_t stream) {
     configured = true;
   }
   dim3 grid((a.dv + kScanCols - 1) / kScanCols, a.H, n_seq);
-  kern<<<grid, kScanThreads, bytes, stream>>>(a, vec);
+  kern<<<grid, ScanTok<DP>::kThreads, bytes, stream>>>(a, vec);
   return launch_status();
 }
 
@@ -305,16 +365,10 @@ int dispatch_scan(const ScanArgs& a, int n_seq, cudaStream_t stream) {
   constexpr int per = 16 / sizeof(T);
   const int v = a.d % per == 0 && a.dv % per == 0 && a.d % 4 == 0 && a.ldq % per == 0 && a.ldk % per == 0 &&
                 a.ldv % per == 0 && aligned_to(a.q, 16) && aligned_to(a.k, 16) && aligned_to(a.v, 16) && aligned_to(a.g, 16);
-  switch ((a.d + 31) / 32) {
-    case 1: return launch_scan<MODE, T, 1>(a, n_seq, v, stream);
-    case 2: return launch_scan<MODE, T, 2>(a, n_seq, v, stream);
-    case 3: return launch_scan<MODE, T, 3>(a, n_seq, v, stream);
-    case 4: return launch_scan<MODE, T, 4>(a, n_seq, v, stream);
-    case 5: return launch_scan<MODE, T, 5>(a, n_seq, v, stream);
-    case 6: return launch_scan<MODE, T, 6>(a, n_seq, v, stream);
-    case 7: return launch_scan<MODE, T, 7>(a, n_seq, v, stream);
-    case 8: return launch_scan<MODE, T, 8>(a, n_seq, v, stream);
-  }
+  if (a.d <= 32) return launch_scan<MODE, T, 32>(a, n_seq, v, stream);
+  if (a.d <= 64) return launch_scan<MODE, T, 64>(a, n_seq, v, stream);
+  if (a.d <= 128) return launch_scan<MODE, T, 128>(a, n_seq, v, stream);
+  if (a.d <= 256) return launch_scan<MODE, T, 256>(a, n_seq, v, stream);
   return -2;
 }
 
@@ -393,12 +447,21 @@ __global__ void delta_inputs_kernel(const DeltaInArgs p) {
     const bool past = tail != nullptr && p.pos0[s] > 0;
     constexpr int kReach = NT > 0 ? NT - 1 : kConvTok;
     float w[kReach + kConvTok];                           // inputs t0 - kReach .. t0 + 15
+    if (t0 - kReach >= sa) {                              // the usual case: all loads at once, no branches
+      const T* xp = x + (size_t)(t0 - kReach) * p.ldx;
+      T raw[kReach + kConvTok];
 #pragma unroll
-    for (int i = 0; i < kReach + kConvTok; ++i) {
-      const int t = t0 - kReach + i;
-      w[i] = 0.f;
-      if (t >= sa) w[i] = to_f<T>(x[(size_t)min(t, t1 - 1) * p.ldx]);
-      else if (past && t >= sa - n1) w[i] = to_f<T>(tail[n1 + t - sa]);
+      for (int i = 0; i < kReach + kConvTok; ++i) raw[i] = xp[(size_t)min(i, t1 - 1 - t0 + kReach) * p.ldx];
+#pragma unroll
+      for (int i = 0; i < kReach + kConvTok; ++i) w[i] = to_f<T>(raw[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kReach + kConvTok; ++i) {
+        const int t = t0 - kReach + i;
+        w[i] = 0.f;
+        if (t >= sa) w[i] = to_f<T>(x[(size_t)min(t, t1 - 1) * p.ldx]);
+        else if (past && t >= sa - n1) w[i] = to_f<T>(tail[n1 + t - sa]);
+      }
     }
 #pragma unroll
     for (int j = 0; j <= kReach; ++j) {                   // tap of the input j tokens back
