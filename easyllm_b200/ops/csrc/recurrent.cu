@@ -5,13 +5,13 @@
 // A state matrix S [d key rows x dv value columns] of one head evolves column by column without mixing columns:
 //   time mixing   o_j = sum_i r_i (S_ij + u_i k_i v_j),          S_ij <- w_i S_ij + k_i v_j
 //   delta rule    S_ij <- g_i S_ij,  e_j = beta (v_j - sum_i k_i S_ij),  S_ij <- S_ij + k_i e_j,  o_j = sum_i q_i S_ij
-// so a CTA owns 32 columns of one (sequence, head) and no CTA waits for another.  A thread keeps 4 columns x 4 or 8 key
-// rows in registers for the whole sequence (8 to 32 lanes share the columns): every operand word read from shared memory
-// then serves four columns, which matters because filling registers from shared memory, not the arithmetic, is what
-// limits a scan.  Both sums of the delta rule are taken from the decayed state at once
+// so a CTA owns 32 columns of one (sequence, head) and no CTA waits for another.  A thread keeps 2 or 4 columns x 4 or
+// 8 key rows in registers for the whole sequence (8 to 32 lanes share the columns): every operand word read from shared
+// memory then serves several columns, which matters because filling registers from shared memory would otherwise limit
+// a scan; with too many columns in a thread the latency of its chain does.  Both sums of the delta rule are taken from the decayed state at once
 // (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the token-to-token chain; the sums of
 // the thread's columns are reduced together, halving the number of values with every step.
-// Consumer warps run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Four more warps copy the operands of the coming
+// Consumer warps run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Eight more warps, one per token of a stage, copy the operands of the coming
 // tokens into a ring of shared-memory stages with cp.async (three stages ahead), convert bf16 operands to fp32, compute
 // the per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous tokens' outputs.
 #include "vec.cuh"
@@ -21,7 +21,7 @@ namespace ell {
 constexpr int kScanCols = 32;         // value columns of a CTA
 constexpr int kScanTok = 8;           // tokens per stage
 constexpr int kScanRing = 4;
-constexpr int kLoadWarps = 4;
+constexpr int kLoadWarps = kScanTok;   // one token of a stage each
 
 enum ScanMode { kWkv = 0, kDelta = 1 };
 
@@ -59,25 +59,30 @@ __device__ __forceinline__ float sum2(f32x2 a) {
   return lo + hi;
 }
 
-// One warp copies n elements; vec: 16-byte pieces (start and length multiples of 16 bytes), else 4-byte ones (fp32).
-template <typename T>
+// One warp copies n <= N elements; vec: 16-byte pieces (start and length multiples of 16 bytes), else 4-byte ones (fp32).
+template <typename T, int N>
 __device__ __forceinline__ void warp_copy(T* dst, const T* src, int n, bool vec, int lane) {
+  constexpr int kPer = 16 / sizeof(T);
   if (vec) {
-    constexpr int kPer = 16 / sizeof(T);
-    for (int c = lane * kPer; c < n; c += 32 * kPer) cp_async16(dst + c, src + c);
+#pragma unroll
+    for (int b = 0; b < N; b += 32 * kPer) {
+      const int c = b + lane * kPer;
+      if (c < n) cp_async16(dst + c, src + c);
+    }
   } else if (sizeof(T) == 4) {
     for (int c = lane; c < n; c += 32) cp_async4(dst + c, src + c);
   }
 }
 
 // Thread layout for heads of up to DP key rows (32, 64, 128 or 256): kLanes lanes hold the rows 4 l + 4 kLanes j .. + 3
-// (j < kJ) of four columns.  Token record the recurrence reads: q | k | g | v | scalar, beta (fp32).  Raw bf16 record:
+// (j < kJ) of kCols columns.  Token record the recurrence reads: q | k | g | v | scalar, beta (fp32).  Raw bf16 record:
 // g | beta (fp32), q | k | v.
 template <int DP>
 struct ScanTok {
   static constexpr int kLanes = DP <= 64 ? 8 : DP / 8;
   static constexpr int kJ = DP / (4 * kLanes);
-  static constexpr int kWarpCols = 4 * (32 / kLanes);
+  static constexpr int kCols = DP <= 128 ? 2 : 4;
+  static constexpr int kWarpCols = kCols * (32 / kLanes);
   static constexpr int kWarps = kScanCols / kWarpCols;             // consumer warps
   static constexpr int kThreads = (kWarps + kLoadWarps) * 32;
   static constexpr int kFloats = 3 * DP + kScanCols + 4;
@@ -118,7 +123,7 @@ __device__ __forceinline__ float reduce_columns(float* v, int l) {
 template <int MODE, typename T, int DP>
 __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanArgs a, int vec) {
   using R = ScanTok<DP>;
-  constexpr int TF = R::kFloats, L = R::kLanes, J = R::kJ;
+  constexpr int TF = R::kFloats, L = R::kLanes, J = R::kJ, NC = R::kCols;
   constexpr bool kF32 = sizeof(T) == 4;
   constexpr int kBufs = kF32 ? kScanRing : 2;          // fp32 records: the ring itself, or two converted stages
   extern __shared__ __align__(16) float sm[];
@@ -133,15 +138,15 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
   const bool loader = warp >= R::kWarps;
   const int lw = warp - R::kWarps;                     // loader warp
   const int l = lane % L;                              // row slice
-  const int cl = warp * R::kWarpCols + lane / L * 4;   // first of the thread's columns within the CTA
+  const int cl = warp * R::kWarpCols + lane / L * NC;  // first of the thread's columns within the CTA
 
   // the copies never write past d and dv: what lies behind must read as zero
   for (int i = threadIdx.x; i < scan_smem_bytes<T, DP>() / 16; i += R::kThreads)
     reinterpret_cast<uint4*>(sm)[i] = make_uint4(0, 0, 0, 0);
 
-  f32x2 S[4][2 * J];                                   // [column][pair of rows]
+  f32x2 S[NC][2 * J];                                  // [column][pair of rows]
 #pragma unroll
-  for (int c = 0; c < 4; ++c)
+  for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int i = 0; i < 2 * J; ++i) S[c][i] = 0ull;
   const int sp = (a.d + 31) / 32 * 32;                 // row stride of the stored state
@@ -150,7 +155,7 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
     srow = a.state + (((size_t)a.slots[s] * a.H + h) * a.dv + col0 + cl) * sp + l * 4;
     if (a.pos0[s] > 0) {
 #pragma unroll
-      for (int c = 0; c < 4; ++c)
+      for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int j = 0; j < J; ++j)
           if (col0 + cl + c < a.dv && l * 4 + j * 4 * L < sp) {
@@ -162,77 +167,79 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
   }
   __syncthreads();
 
-  auto issue = [&](int ch) {                           // start the copies of a chunk (this warp's tokens)
-    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
-      const size_t t = (size_t)t_begin + ch * kScanTok + i;
-      const T* qp = reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
-      const T* kp = reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
-      const T* vp = reinterpret_cast<const T*>(a.v) + t * a.ldv + (size_t)h * a.dv + col0;
-      const int nv = min(kScanCols, a.dv - col0);
+  // loader warp lw owns token lw of every stage
+  const size_t t_mine = (size_t)t_begin + lw;
+  const T* q_src = reinterpret_cast<const T*>(a.q) + t_mine * a.ldq + (size_t)hk * a.d;
+  const T* k_src = reinterpret_cast<const T*>(a.k) + t_mine * a.ldk + (size_t)hk * a.d;
+  const T* v_src = reinterpret_cast<const T*>(a.v) + t_mine * a.ldv + (size_t)h * a.dv + col0;
+  const float* g_src = a.g + (t_mine * a.H + h) * a.d;
+  const float* b_src = MODE == kDelta ? a.beta + t_mine * a.H + h : nullptr;
+  float* o_dst = a.o + (t_mine * a.H + h) * a.dv + col0 + lane;
+  const size_t g_step = (size_t)kScanTok * a.H * a.d, o_step = (size_t)kScanTok * a.H * a.dv;
+  const int nv = min(kScanCols, a.dv - col0);
+  float u[DP / 32];                                    // wkv: the bonus of the loader lane's channels
+#pragma unroll
+  for (int c = 0; c < DP / 32; ++c)
+    u[c] = MODE == kWkv && loader && c * 32 + lane < a.d ? a.u[(size_t)h * a.d + c * 32 + lane] : 0.f;
+
+  auto issue = [&](int ch) {                           // start the copies of a stage
+    if (ch * kScanTok + lw < n_tok) {
       float *gd, *bd;
       T *qd, *kd, *vd;
       if (kF32) {
-        float* tok = sm + ((ch % kScanRing) * kScanTok + i) * TF;
+        float* tok = sm + ((ch % kScanRing) * kScanTok + lw) * TF;
         qd = reinterpret_cast<T*>(tok), kd = qd + DP, gd = tok + 2 * DP, vd = reinterpret_cast<T*>(tok + 3 * DP);
         bd = tok + 3 * DP + kScanCols + 1;
       } else {
-        uint8_t* rec = raw + ((ch % kScanRing) * kScanTok + i) * R::kRawBytes;
+        uint8_t* rec = raw + ((ch % kScanRing) * kScanTok + lw) * R::kRawBytes;
         gd = reinterpret_cast<float*>(rec), bd = gd + DP, qd = reinterpret_cast<T*>(gd + DP + 4), kd = qd + DP, vd = kd + DP;
       }
-      warp_copy<T>(qd, qp, a.d, vec, lane);
-      warp_copy<T>(kd, kp, a.d, vec, lane);
-      warp_copy<float>(gd, a.g + (t * a.H + h) * a.d, a.d, vec, lane);
-      warp_copy<T>(vd, vp, nv, vec, lane);
-      if (MODE == kDelta && lane == 0) cp_async4(bd, a.beta + t * a.H + h);
+      const size_t t = (size_t)ch * kScanTok;
+      warp_copy<T, DP>(qd, q_src + t * a.ldq, a.d, vec, lane);
+      warp_copy<T, DP>(kd, k_src + t * a.ldk, a.d, vec, lane);
+      warp_copy<float, DP>(gd, g_src + ch * g_step, a.d, vec, lane);
+      warp_copy<T, kScanCols>(vd, v_src + t * a.ldv, nv, vec, lane);
+      if (MODE == kDelta && lane == 0) cp_async4(bd, b_src + t * a.H);
     }
     cp_async_commit();
   };
-  auto prepare = [&](int ch) {                         // a landed chunk: scalars, and fp32 records of bf16 operands
+  auto prepare = [&](int ch) {                         // a landed stage: scalars, and fp32 records of bf16 operands
     cp_async_wait<kScanRing - 2>();
     __syncwarp();
-    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
-      const size_t t = (size_t)t_begin + ch * kScanTok + i;
-      float* tok = sm + ((ch % kBufs) * kScanTok + i) * TF;
-      float dot = 0.f;
-      if (kF32) {
+    if (ch * kScanTok + lw >= n_tok) return;
+    float* tok = sm + ((ch % kBufs) * kScanTok + lw) * TF;
+    float dot = 0.f;
+    if (kF32) {
 #pragma unroll
-        for (int c = 0; c < DP / 32; ++c) {
-          const int x = c * 32 + lane;
-          const float p = tok[x] * tok[DP + x];
-          dot += MODE == kWkv ? (x < a.d ? p * a.u[(size_t)h * a.d + x] : 0.f) : p;
-        }
-      } else {
-        const uint8_t* rec = raw + ((ch % kScanRing) * kScanTok + i) * R::kRawBytes;
-        const float* gs = reinterpret_cast<const float*>(rec);
-        const T* qs = vec ? reinterpret_cast<const T*>(gs + DP + 4)
-                          : reinterpret_cast<const T*>(a.q) + t * a.ldq + (size_t)hk * a.d;
-        const T* ks = vec ? reinterpret_cast<const T*>(gs + DP + 4) + DP
-                          : reinterpret_cast<const T*>(a.k) + t * a.ldk + (size_t)hk * a.d;
-        const T* vs = vec ? reinterpret_cast<const T*>(gs + DP + 4) + 2 * DP
-                          : reinterpret_cast<const T*>(a.v) + t * a.ldv + (size_t)h * a.dv + col0;
-#pragma unroll
-        for (int c = 0; c < DP / 32; ++c) {
-          const int x = c * 32 + lane;
-          const bool in = x < a.d;
-          const float q = in ? to_f<T>(qs[x]) : 0.f, k = in ? to_f<T>(ks[x]) : 0.f;
-          tok[x] = q;
-          tok[DP + x] = k;
-          tok[2 * DP + x] = gs[x];
-          dot += MODE == kWkv ? (in ? q * k * a.u[(size_t)h * a.d + x] : 0.f) : q * k;
-        }
-        tok[3 * DP + lane] = col0 + lane < a.dv ? to_f<T>(vs[lane]) : 0.f;
-        if (lane == 0) tok[3 * DP + kScanCols + 1] = gs[DP];
+      for (int c = 0; c < DP / 32; ++c) {
+        const float p = tok[c * 32 + lane] * tok[DP + c * 32 + lane];
+        dot = MODE == kWkv ? fmaf(p, u[c], dot) : dot + p;
       }
-      dot = warp_sum(dot);
-      if (lane == 0) tok[3 * DP + kScanCols] = dot;
+    } else {
+      const float* gs = reinterpret_cast<const float*>(raw + ((ch % kScanRing) * kScanTok + lw) * R::kRawBytes);
+      const size_t t = (size_t)ch * kScanTok;
+      const T* qs = vec ? reinterpret_cast<const T*>(gs + DP + 4) : q_src + t * a.ldq;
+      const T* ks = vec ? reinterpret_cast<const T*>(gs + DP + 4) + DP : k_src + t * a.ldk;
+      const T* vs = vec ? reinterpret_cast<const T*>(gs + DP + 4) + 2 * DP : v_src + t * a.ldv;
+#pragma unroll
+      for (int c = 0; c < DP / 32; ++c) {
+        const int x = c * 32 + lane;
+        const bool in = x < a.d;
+        const float q = in ? to_f<T>(qs[x]) : 0.f, k = in ? to_f<T>(ks[x]) : 0.f;
+        tok[x] = q;
+        tok[DP + x] = k;
+        tok[2 * DP + x] = gs[x];
+        dot = MODE == kWkv ? fmaf(q * k, u[c], dot) : fmaf(q, k, dot);
+      }
+      tok[3 * DP + lane] = lane < nv ? to_f<T>(vs[lane]) : 0.f;
+      if (lane == 0) tok[3 * DP + kScanCols + 1] = gs[DP];
     }
+    dot = warp_sum(dot);
+    if (lane == 0) tok[3 * DP + kScanCols] = dot;
   };
   auto store = [&](int ch) {
-    const float* ob = outb + (ch & 1) * kScanTok * kScanCols;
-    for (int i = lw; i < min(kScanTok, n_tok - ch * kScanTok); i += kLoadWarps) {
-      const size_t t = (size_t)t_begin + ch * kScanTok + i;
-      if (col0 + lane < a.dv) a.o[(t * a.H + h) * a.dv + col0 + lane] = ob[i * kScanCols + lane];
-    }
+    if (ch * kScanTok + lw < n_tok && lane < nv)
+      o_dst[ch * o_step] = outb[((ch & 1) * kScanTok + lw) * kScanCols + lane];
   };
 
   if (loader) {
@@ -251,7 +258,8 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
       const int cnt = min(kScanTok, n_tok - ch * kScanTok);
       float* ob = outb + (ch & 1) * kScanTok * kScanCols;
       // after the reduction a lane holds the sum of one column (and, in the delta rule, of k or of q)
-      constexpr int kC1 = MODE == kDelta ? L / 4 : L / 2, kC0 = kC1 / 2;
+      constexpr int kTop = MODE == kDelta ? L / 4 : L / 2;            // lane bits: k or q | column, high bit first
+      constexpr int kC0 = NC == 4 ? kTop / 2 : kTop, kC1 = NC == 4 ? kTop : 0;
       const int my_c = (l & kC1 ? 2 : 0) + (l & kC0 ? 1 : 0);
       const bool is_q = MODE == kWkv || (l & (L / 2));
       const bool writes = is_q && (l & (kC0 - 1)) == 0;
@@ -267,12 +275,11 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
           g[j] = *reinterpret_cast<const ulonglong2*>(tok + 2 * DP + j * 4 * L + l * 4);
         }
         if (MODE == kWkv) {
-          const float4 v4 = *reinterpret_cast<const float4*>(tok + 3 * DP + cl);
-          const float v[4] = {v4.x, v4.y, v4.z, v4.w};
-          float sum[4];
+          float sum[NC];
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            const f32x2 vv = pack2(v[c], v[c]);
+          for (int c = 0; c < NC; ++c) {
+            const float v = tok[3 * DP + cl + c];
+            const f32x2 vv = pack2(v, v);
             f32x2 o = 0ull;
 #pragma unroll
             for (int j = 0; j < J; ++j) {
@@ -283,12 +290,12 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
             }
             sum[c] = sum2(o);
           }
-          return fmaf(sc, v_mine, reduce_columns<4, L>(sum, l));
+          return fmaf(sc, v_mine, reduce_columns<NC, L>(sum, l));
         } else {
           const float beta = tok[3 * DP + kScanCols + 1];
-          float sum[8];
+          float sum[2 * NC];
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < NC; ++c) {
             f32x2 ks = 0ull, qs = 0ull;
 #pragma unroll
             for (int j = 0; j < J; ++j) {
@@ -300,12 +307,12 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
               qs = fma2(q[j].y, S[c][2 * j + 1], qs);
             }
             sum[c] = sum2(ks);
-            sum[4 + c] = sum2(qs);
+            sum[NC + c] = sum2(qs);
           }
-          const float mine = reduce_columns<8, L>(sum, l);
+          const float mine = reduce_columns<2 * NC, L>(sum, l);
           const float e = beta * (v_mine - mine);      // of the lanes that hold a k sum
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < NC; ++c) {
             const float ec = __shfl_sync(0xffffffffu, e, (lane & ~(L - 1)) + (c & 2 ? kC1 : 0) + (c & 1 ? kC0 : 0));
             const f32x2 ee = pack2(ec, ec);
 #pragma unroll
@@ -336,7 +343,7 @@ __global__ void __launch_bounds__(ScanTok<DP>::kThreads) scan_kernel(const ScanA
     store(n_chunk - 1);
   } else if (srow != nullptr) {
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
       for (int j = 0; j < J; ++j)
         if (col0 + cl + c < a.dv && l * 4 + j * 4 * L < sp)
