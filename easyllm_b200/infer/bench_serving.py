@@ -31,9 +31,9 @@ def pafodra_config(s):
     wkv = {"type": "wkv", "mixer": {"heads": s["width"] // 64, "dim": 64}}
     delta = {"type": "channel_delta", "mixer": {"heads": s["rheads"], "kv_heads": s["rheads"], "dim": d, "vdim": d, "conv": 4},
              "mlp": moe}
-    period = [att, dict(wkv, mlp=moe), dict(wkv, mlp={"kind": "dense", "ff": s["ff"]}), delta, att]
+    period = [dict(wkv, mlp=moe), att, delta, att, dict(wkv, mlp={"kind": "dense", "ff": s["ff"]})]
     return {"architecture": "Pafodra", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
-            "embedding": {"scale": 16.0}, "layers": [period[i % 5] for i in range(s["layers"])]}
+            "embedding": {"scale": 4.0}, "layers": [period[i % 5] for i in range(s["layers"])]}
 
 
 def build(which, s):
