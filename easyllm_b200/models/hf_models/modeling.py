@@ -574,7 +574,8 @@ class CausalLM(nn.Module):
         every new token.  ``attention_mask``: rows of unequal length (padding on either side of ``input_ids``; new
         tokens are appended after column ``s``).  A row ends at ``eos_token_id`` or when its tail equals one of
         ``stop_words_ids`` (token sequences; the stop sequence stays in the output, later positions are filled with eos).
-        ``cuda_graph``: on a GPU, replay the decode step as a CUDA graph once it has run eagerly.
+        ``cuda_graph``: on a GPU, replay the decode step as a CUDA graph once it has run eagerly (not with dynamic NTK,
+        whose tables depend on the length, nor with the 8-bit cache).
         ``soft_prefix``: ``{"embeds": [P, hidden]}`` (prompt tuning: virtual input embeddings in front of the
         prompt) or ``{"kv": [layers, 2, P, kv_heads, head_dim]}`` (prefix tuning: pre-filled cache entries)."""
         from ...infer.generation import sample_next
@@ -624,7 +625,7 @@ class CausalLM(nn.Module):
             else:
                 logits = self.logits(self.step(state, slots, toks[:, -1])[0])
                 if cuda_graph and dev.type == "cuda" and dt != torch.float16 and not a.use_cache_quantization and \
-                        max_new_tokens - step > 4:
+                        a.rope_dynamic_ntk_max_pos is None and max_new_tokens - step > 4:
                     graph = DecodeGraph(self, state, slots)
             if repetition_penalty != 1.0:
                 seen = torch.gather(logits, 1, toks)

@@ -8,12 +8,13 @@
 // so a CTA owns 32 columns of one (sequence, head) and no CTA waits for another.  A thread keeps 2 or 4 columns x 4 or
 // 8 key rows in registers for the whole sequence (8 to 32 lanes share the columns): every operand word read from shared
 // memory then serves several columns, which matters because filling registers from shared memory would otherwise limit
-// a scan; with too many columns in a thread the latency of its chain does.  Both sums of the delta rule are taken from the decayed state at once
-// (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the token-to-token chain; the sums of
-// the thread's columns are reduced together, halving the number of values with every step.
-// Consumer warps run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Eight more warps, one per token of a stage, copy the operands of the coming
-// tokens into a ring of shared-memory stages with cp.async (three stages ahead), convert bf16 operands to fp32, compute
-// the per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous tokens' outputs.
+// a scan; with too many columns in a thread the latency of its chain does.  Both sums of the delta rule are taken from
+// the decayed state at once (o_j = sum_i q_i g_i S_ij + (q . k) e_j), which leaves one shuffle reduction on the
+// token-to-token chain; the sums of the thread's columns are reduced together, halving the number of values with every
+// step.  Consumer warps run the recurrence on packed fp32 pairs (fma.rn.f32x2).  Eight more warps, one per token of a
+// stage, copy the operands of the coming tokens into a ring of shared-memory stages with cp.async (three stages ahead),
+// convert bf16 operands to fp32, compute the per-token scalars (q . k, or sum_i r_i u_i k_i), and write the previous
+// tokens' outputs.
 #include "vec.cuh"
 
 namespace ell {

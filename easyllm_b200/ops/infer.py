@@ -37,11 +37,12 @@ def no_grad_check(*ts):
 
 def make_adjacent_(params):
     """Move parameters of one group back to back into one storage, so that ``fused`` aliases them without a copy.
-    Parameters with an fp32 ``main_grad`` belong to an optimizer's flat buffer and are left where they are."""
+    Parameters that live in a larger buffer (an optimizer's flat one) are left where they are."""
     if len(params) < 2 or any(getattr(p, "main_grad", None) is not None for p in params) or fused_alias(params) is not None:
         return
-    if len({(p.dtype, p.device) for p in params}) != 1:
-        return
+    if len({(p.dtype, p.device) for p in params}) != 1 or \
+            any(p.untyped_storage().nbytes() != p.numel() * p.element_size() for p in params):
+        return                                          # a view of somebody's larger buffer stays where it is
     flat = torch.cat([p.detach().reshape(-1) for p in params])
     at = 0
     for p in params:
