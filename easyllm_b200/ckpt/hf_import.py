@@ -68,18 +68,31 @@ for _p in ("gate", "up", "down"):
     PAFODRA_NAMES[f"mlp.{_p}"], PAFODRA_NAMES[f"mlp.{_p}.b"] = f"mlp.{_p}_proj.weight", f"mlp.{_p}_proj.bias"
 PAFODRA_NAMES.update({"mlp.router": "mlp.router.weight", "mlp.shared.up": "mlp.shared.up_proj.weight",
                       "mlp.shared.down": "mlp.shared.down_proj.weight", "mlp.shared.sg": "mlp.shared_gate.weight"})
-_PAFODRA_RULES = [(rf"^l(\d+)\.{re.escape(k)}$", rf"\1:{v}") for k, v in PAFODRA_NAMES.items()] + [
+# Megozen, likewise
+MEGOZEN_NAMES = {"norm1": "input_layernorm.weight", "norm2": "mlp_layernorm.weight", "mix.dkv.norm": "mixer.dkv_norm",
+                 "mlp.router": "mlp.router.weight", "mlp.router.b": "mlp.router_bias"}
+MEGOZEN_NAMES.update({f"mix.{p}": f"mixer.{p}_proj.weight" for p in ("q", "dkv", "uk", "uv", "g", "o")})
+MEGOZEN_NAMES.update({f"mlp.shared.{p}": f"mlp.shared.{p}_proj.weight" for p in ("gate", "up", "down")})
+HYBRID_NAMES = {"pafodra": PAFODRA_NAMES, "megozen": MEGOZEN_NAMES}
+
+
+def _hybrid_rules(names, more):
+    return [(rf"^l(\d+)\.{re.escape(k)}$", rf"\1:{v}") for k, v in names.items()] + [
+        (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"\1:mlp.experts.\2.\3"),
+        (r"^embed$", "embed:word_embeddings.weight"),
+        (r"^head$", "head:word_embeddings.weight"),
+        (r"^final\.norm$", "norm:weight")] + more
+
+
+_PAFODRA_RULES = _hybrid_rules(PAFODRA_NAMES, [
     (r"^l(\d+)\.mix\.mu\.([rkvgw])$", r"\1:mixer.mu.\2"),
-    (r"^l(\d+)\.mlp\.e(\d+)\.(up|down)$", r"\1:mlp.experts.\2.\3"),
-    (r"^embed$", "embed:word_embeddings.weight"),
-    (r"^head$", "head:word_embeddings.weight"),
-    (r"^final\.norm$", "norm:weight"),
     (r"^final\.norm\.b$", "norm:bias"),
     (r"^final\.norm\.alpha$", "norm:alpha"),
-]
+])
+_MEGOZEN_RULES = _hybrid_rules(MEGOZEN_NAMES, [(r"^bigram$", "embed:pairs")])
 RULES = {"llama": _LLAMA_RULES, "llama_pack": _LLAMA_RULES, "qwen": _QWEN_RULES,
          "internlm2": _INTERNLM2_RULES, "internlm2_pack": _INTERNLM2_RULES, "baichuan": _LLAMA_RULES,
-         "internlm": _LLAMA_RULES, "pafodra": _PAFODRA_RULES}
+         "internlm": _LLAMA_RULES, "pafodra": _PAFODRA_RULES, "megozen": _MEGOZEN_RULES}
 
 
 def canonicalize(hf_state: Dict[str, torch.Tensor], pretrain_type: str, n_heads: int, n_kv_heads: int,

@@ -3,8 +3,8 @@
 ``MODULE_ZOO_REGISTRY`` names kept: ``LlamaForCausalLM``, ``InternLMForCausalLM``,
 ``InternLM2ForCausalLM``, ``BaiChuanForCausalLM``, ``BaiChuan2ForCausalLM``,
 ``BaiChuan2ForCausalLM13B``, ``QWenForCausalLM``, ``QWenForVL``, ``KVLlamaForCausalLM``,
-``medusa`` (llm/models/hf_models/*/__init__.py).  Added: ``PafodraForCausalLM`` (hybrid attention / recurrent decoder,
-inference only) and ``AutoCausalLM`` (family from the checkpoint's ``config.json``).  ``get_model_cfg`` mirrors
+``medusa`` (llm/models/hf_models/*/__init__.py).  Added: ``PafodraForCausalLM`` (hybrid attention / recurrent decoder)
+and ``MegozenForCausalLM`` (latent attention and gated experts in parallel blocks), both inference only, and ``AutoCausalLM`` (family from the checkpoint's ``config.json``).  ``get_model_cfg`` mirrors
 utils/model_utils.py:6-70: ``model_name_or_path``, ``torch_dtype``; the private
 ``_flash_*_2_enabled`` switches are accepted and ignored (the fused kernels are always on).
 A config may give ``arch`` (a dict of HFArch fields) instead of a path to build a
@@ -46,7 +46,8 @@ def _builder(family):
 for _name, _fam in (("LlamaForCausalLM", "llama"), ("KVLlamaForCausalLM", "llama"), ("InternLMForCausalLM", "internlm"),
                     ("InternLM2ForCausalLM", "internlm2"), ("BaiChuanForCausalLM", "baichuan"),
                     ("BaiChuan2ForCausalLM", "baichuan2"), ("BaiChuan2ForCausalLM13B", "baichuan2-13b"),
-                    ("QWenForCausalLM", "qwen"), ("PafodraForCausalLM", "pafodra"), ("AutoCausalLM", None)):
+                    ("QWenForCausalLM", "qwen"), ("PafodraForCausalLM", "pafodra"), ("MegozenForCausalLM", "megozen"),
+                    ("AutoCausalLM", None)):
     MODULE_ZOO_REGISTRY.register(_name, _builder(_fam))
 
 from . import medusa as _medusa  # noqa: E402,F401

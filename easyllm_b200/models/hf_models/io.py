@@ -9,9 +9,11 @@ from __future__ import annotations
 import torch
 
 from ...ckpt.hf_import import canonicalize
+from .feedforward import SparseGLU
 
 _FAMILY_RULES = {"llama": "llama", "internlm": "llama", "baichuan": "baichuan", "baichuan2": "baichuan",
-                 "baichuan2-13b": "baichuan", "internlm2": "internlm2", "qwen": "qwen", "pafodra": "pafodra"}
+                 "baichuan2-13b": "baichuan", "internlm2": "internlm2", "qwen": "qwen", "pafodra": "pafodra",
+                 "megozen": "megozen"}
 _MIXES = "rkvgw"          # rows of TimeMix.mu
 
 
@@ -22,7 +24,7 @@ def import_state(hf_state, arch):
     for slot, tensors in canon.items():
         for name, t in tensors.items():
             if slot == "embed":
-                out["model.embed_tokens.weight"] = t
+                out["model.embed_pairs.weight" if name == "pairs" else "model.embed_tokens.weight"] = t
             elif slot == "norm":
                 out[f"model.norm.{name}"] = t
             elif slot == "head":
@@ -53,8 +55,13 @@ def _stack_hybrid(sd, arch):
         mine = {k[len(src):]: v for k, v in sd.items() if k.startswith(src)}
         if spec.type == "wkv":
             mine["mixer.mu"] = torch.stack([mine.pop(f"mixer.mu.{c}") for c in _MIXES])
+        if spec.mlp is None:
+            mine.pop("mlp_layernorm.weight", None)          # the norm of a feed-forward that is not there
         if spec.mlp is not None and spec.mlp["kind"] == "moe":
-            for p in ("up", "down"):
+            if arch.expert_form == "glu":
+                mine["mlp.experts_gate_up"] = torch.stack([SparseGLU.blocked(*(mine.pop(f"mlp.experts.{e}.{p}") for p in ("gate", "up")))
+                                                           for e in range(spec.mlp["router"]["experts"])])
+            for p in ("down",) if arch.expert_form == "glu" else ("up", "down"):
                 mine[f"mlp.experts_{p}"] = torch.stack([mine.pop(f"mlp.experts.{e}.{p}")
                                                         for e in range(spec.mlp["router"]["experts"])])
         out.update({dst + k: v for k, v in mine.items()})
@@ -62,13 +69,16 @@ def _stack_hybrid(sd, arch):
     return out
 
 
-def _export_pafodra(sd, arch):
+def _export_hybrid(sd, arch):
     from .modeling import weight_owner
-    from ...ckpt.hf_import import PAFODRA_NAMES
-    back = {v: k for k, v in PAFODRA_NAMES.items()}
+    from ...ckpt.hf_import import HYBRID_NAMES
+    back = {v: k for k, v in HYBRID_NAMES[arch.family].items()}
     out = {"embed": sd["model.embed_tokens.weight"], "head": sd["lm_head.weight"]}
+    if arch.bigram is not None:
+        out["bigram"] = sd["model.embed_pairs.weight"]
     for n, suffix in (("weight", ""), ("bias", ".b"), ("alpha", ".alpha")):
-        out["final.norm" + suffix] = sd["model.norm." + n]
+        if "model.norm." + n in sd:
+            out["final.norm" + suffix] = sd["model.norm." + n]
     for i in range(len(arch.layers)):
         if weight_owner(arch.layers, i) != i:
             continue
@@ -79,6 +89,9 @@ def _export_pafodra(sd, arch):
             name = k[len(pre):]
             if name == "mixer.mu":
                 out.update({f"l{i}.mix.mu.{c}": v[j] for j, c in enumerate(_MIXES)})
+            elif name == "mlp.experts_gate_up":
+                for e, w in enumerate(v):
+                    out[f"l{i}.mlp.e{e}.gate"], out[f"l{i}.mlp.e{e}.up"] = SparseGLU.split(w)
             elif name in ("mlp.experts_up", "mlp.experts_down"):
                 out.update({f"l{i}.mlp.e{e}.{name[12:]}": w for e, w in enumerate(v)})
             else:
@@ -91,8 +104,8 @@ def export_state(sd, arch):
     fam = arch.family
     if fam in ("llama", "internlm"):
         return sd
-    if fam == "pafodra":
-        return _export_pafodra(sd, arch)
+    if arch.layers is not None:
+        return _export_hybrid(sd, arch)
     out = {}
     L = arch.num_hidden_layers
     hq, hk, d, h = arch.num_attention_heads, arch.kv_heads, arch.head_dim, arch.hidden_size
@@ -144,13 +157,14 @@ def export_state(sd, arch):
 
 def export_config(arch):
     a = arch
-    if a.family == "pafodra":
+    if a.layers is not None:
         layers = []
         for l in a.layers:
-            e = {"type": l.type, "mixer": {k: v for k, v in l.mixer.items() if not k.endswith("_rank")}, "mlp": l.mlp}
+            e = {"type": l.type, "mixer": {k: v for k, v in l.mixer.items() if k not in ("decay_rank", "gate_rank")}, "mlp": l.mlp}
             layers.append(e if l.weights_of is None else dict(e, weights_of=l.weights_of))
-        return {"architecture": "Pafodra", "vocab": a.vocab_size, "width": a.hidden_size, "layers": layers,
-                "norm": {"eps": a.norm_eps}, "embedding": {"scale": a.embedding_scale}}
+        emb = {"scale": a.embedding_scale} if a.family == "pafodra" else {} if a.bigram is None else {"bigram": a.bigram}
+        return {"architecture": a.family.capitalize(), "vocab": a.vocab_size, "width": a.hidden_size, "layers": layers,
+                "norm": {"eps": a.norm_eps}, "embedding": emb}
     if a.family == "qwen":
         return {"model_type": "qwen", "vocab_size": a.vocab_size, "hidden_size": a.hidden_size,
                 "intermediate_size": 2 * a.intermediate_size, "num_hidden_layers": a.num_hidden_layers,

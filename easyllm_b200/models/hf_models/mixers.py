@@ -1,10 +1,11 @@
-"""Token mixers without a key/value cache, and the norm they come with.
+"""Token mixers without a key/value cache, and the norms of the parallel blocks.
 
 Each mixer is built from its sizes (a dict) and is called as ``mixer(h, meta, state, residual)``: ``h [T, hidden]`` are
 the normed inputs of the packed sequences of ``meta``, ``state`` the layer's ``SlotTensors`` (None: every sequence starts
 here and nothing is kept), and the output projection is accumulated into the fp32 stream ``residual``.
 
 * ``DynamicTanh``: the norm ``tanh(alpha x) w + b``.
+* ``LayerNorm``: layer norm without a bias, on the fp32 stream.
 * ``TimeMix``: RWKV-style mixing with a decay per key channel and a bonus for the current token.
 * ``ChannelDelta``: the gated delta rule with a decay per head and key channel, short convolutions on q, k, v.
 """
@@ -32,6 +33,20 @@ class DynamicTanh(nn.Module):
     def forward(self, x, add=None):
         """Norm of ``x``.  ``add [dim]``: after its norm is taken, ``x`` (fp32, updated in place) gains this vector."""
         return iops.dynamic_tanh(x, self.alpha, self.weight, self.bias, self.out_dtype, add)
+
+
+class LayerNorm(nn.Module):
+    """``(x - mean) / sqrt(variance + eps) * w`` in fp32.  ``also``: a second norm of the same ``x``; both come from one
+    pass, and the result is the pair."""
+
+    def __init__(self, dim, eps, dtype):
+        super().__init__()
+        self.weight, self.eps, self.out_dtype = _vec(dim, fill=1.0), eps, dtype
+
+    def forward(self, x, also=None):
+        if also is None:
+            return iops.layer_norms(x, [self.weight], self.eps, self.out_dtype)[0]
+        return iops.layer_norms(x, [self.weight, also.weight], self.eps, self.out_dtype)
 
 
 class TimeMix(nn.Module):

@@ -28,8 +28,9 @@ from ... import ops
 from ...ops import infer as iops
 from ...ops import reference as ref
 from ..layers import RotaryTables, alibi_slopes
-from .feedforward import DenseGLU, SparseMoE
-from .mixers import ChannelDelta, DynamicTanh, TimeMix
+from .feedforward import DenseGLU, SparseGLU, SparseMoE
+from .latent import LatentAttention
+from .mixers import ChannelDelta, DynamicTanh, LayerNorm, TimeMix
 from .state import DecodeGraph, DecodeState, KVRows
 
 
@@ -37,7 +38,7 @@ from .state import DecodeGraph, DecodeState, KVRows
 class LayerSpec:
     """One layer of a decoder whose layers differ: the mixer and its sizes, the feed-forward (None: no feed-forward),
     and ``weights_of``, the layer whose tensors it uses (with a cache or state of its own)."""
-    type: str = "attention"               # attention | wkv | channel_delta
+    type: str = "attention"               # attention | wkv | channel_delta | latent_attention
     mixer: dict = field(default_factory=dict)
     mlp: Optional[dict] = None
     weights_of: Optional[int] = None
@@ -71,8 +72,11 @@ class HFArch:
     # decoders whose layers differ: one spec per layer (None: num_hidden_layers equal attention + SwiGLU layers), run as
     # parallel blocks x + mixer(norm x) + ff(norm x) on an fp32 stream
     layers: Optional[List[LayerSpec]] = None
-    norm_eps: float = 1e-5                # eps of the mixers' own head norms
+    norm_eps: float = 1e-5                # eps of the layer norms and of the mixers' own norms
     embedding_scale: float = 1.0
+    block_norm: str = "dynamic_tanh"      # dynamic_tanh: one norm for mixer and ff | layer_norm: one for each
+    expert_form: str = "relu2"            # relu2: two matrices, input weighting | glu: three, softmax weights
+    bigram: Optional[dict] = None         # table of (previous token, token) pairs: buckets, mul_prev, mul_cur
 
     @property
     def kv_heads(self):
@@ -88,6 +92,8 @@ def arch_from_hf_config(cfg: dict, family: Optional[str] = None) -> HFArch:
     mt = (family or cfg.get("model_type") or cfg.get("architecture") or "llama").lower()
     if mt == "pafodra":
         return _pafodra_arch(cfg)
+    if mt == "megozen":
+        return _megozen_arch(cfg)
     a = HFArch(family=mt)
     g = cfg.get
     if mt == "qwen":
@@ -129,14 +135,15 @@ def arch_from_hf_config(cfg: dict, family: Optional[str] = None) -> HFArch:
 
 
 _MIXER_SIZES = {"attention": ("heads", "kv_heads", "dim", "vdim", "scale"), "wkv": ("heads", "dim"),
-                "channel_delta": ("heads", "kv_heads", "dim", "vdim", "conv")}
+                "channel_delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
+                "latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot")}
 
 
-def _pafodra_arch(cfg: dict) -> HFArch:
-    """``config.json`` of a Pafodra model: vocab, width, norm.eps, embedding.scale and one entry per layer."""
+def _layer_specs(cfg: dict, mixers, mlps) -> List[LayerSpec]:
+    """The 'layers' entries of a ``config.json``, checked; ``mixers`` / ``mlps``: the kinds this family has."""
     layers = []
     for i, e in enumerate(cfg["layers"]):
-        if e["type"] not in _MIXER_SIZES:
+        if e["type"] not in mixers:
             raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
         missing = [k for k in _MIXER_SIZES[e["type"]] if k not in e["mixer"]]
         if missing:
@@ -145,12 +152,34 @@ def _pafodra_arch(cfg: dict) -> HFArch:
         if kv and e["mixer"]["heads"] % kv:
             raise ValueError(f"layer {i}: {e['mixer']['heads']} heads do not divide into {kv} key/value heads")
         mlp = e.get("mlp")
-        if mlp is not None and mlp["kind"] not in ("dense", "moe"):
+        if mlp is not None and mlp["kind"] not in mlps:
             raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
         w = e.get("weights_of")
         if w is not None and not 0 <= w < len(cfg["layers"]):
             raise ValueError(f"layer {i}: weights_of {w} is not a layer")
         layers.append(LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else dict(mlp), w))
+    return layers
+
+
+def _megozen_arch(cfg: dict) -> HFArch:
+    """``config.json`` of a Megozen model: vocab, width, norm.eps, embedding.bigram and one entry per layer."""
+    layers = _layer_specs(cfg, ("latent_attention",), ("moe",))
+    for i, l in enumerate(layers):
+        dims = l.mixer["rot"]["dims"]
+        if dims % 2 or l.mixer["rot_dim"] % 2 or not 0 < dims <= l.mixer["rot_dim"]:
+            raise ValueError(f"layer {i}: {dims} rotated dimensions of {l.mixer['rot_dim']}")
+        if l.mixer.get("mask") and l.mixer["mask"]["size"] < 1:
+            raise ValueError(f"layer {i}: a window of {l.mixer['mask']['size']} tokens")
+    return HFArch(family="megozen", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layers=layers,
+                  num_hidden_layers=len(layers), num_attention_heads=layers[0].mixer["heads"] if layers else 1,
+                  num_key_value_heads=1, norm_eps=cfg["norm"]["eps"], block_norm="layer_norm", expert_form="glu",
+                  bigram=(cfg.get("embedding") or {}).get("bigram"), position="none", bos_token_id=cfg.get("bos_token_id"),
+                  eos_token_id=cfg.get("eos_token_id"), pad_token_id=cfg.get("pad_token_id"))
+
+
+def _pafodra_arch(cfg: dict) -> HFArch:
+    """``config.json`` of a Pafodra model: vocab, width, norm.eps, embedding.scale and one entry per layer."""
+    layers = _layer_specs(cfg, ("attention", "wkv", "channel_delta"), ("dense", "moe"))
     att = next((l.mixer for l in layers if l.type == "attention"), {})
     return HFArch(family="pafodra", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layers=layers,
                   num_hidden_layers=len(layers), num_attention_heads=att.get("heads", 1),
@@ -360,30 +389,40 @@ class DecoderLayer(nn.Module):
         return self.mlp(n2), h
 
 
+def _block_norm(a: HFArch, dtype):
+    return DynamicTanh(a.hidden_size, dtype) if a.block_norm == "dynamic_tanh" else LayerNorm(a.hidden_size, a.norm_eps, dtype)
+
+
 class ParallelLayer(nn.Module):
-    """``x + mixer(h) + ff(h)`` with one norm ``h = norm(x)``: both sublayers accumulate into the fp32 stream ``x``."""
+    """``x + mixer(norm x) + ff(norm x)``: both sublayers accumulate into the fp32 stream ``x``.  They share one norm, or
+    (``block_norm: layer_norm``) have one each, taken from the same ``x`` in one pass."""
 
     def __init__(self, a: HFArch, spec: LayerSpec, dtype):
         super().__init__()
         m = spec.mixer
-        self.input_layernorm = DynamicTanh(a.hidden_size, dtype)
+        self.input_layernorm = _block_norm(a, dtype)
+        self.mlp_layernorm = _block_norm(a, dtype) if a.block_norm == "layer_norm" and spec.mlp is not None else None
         if spec.type == "attention":
             self.mixer = Attention(a, dtype, dict(m, sink=True))
         else:
-            self.mixer = {"wkv": TimeMix, "channel_delta": ChannelDelta}[spec.type](a.hidden_size, m, a.norm_eps, dtype)
+            self.mixer = {"wkv": TimeMix, "channel_delta": ChannelDelta,
+                          "latent_attention": LatentAttention}[spec.type](a.hidden_size, m, a.norm_eps, dtype)
         self.mlp = None
         if spec.mlp is not None:
             self.mlp = DenseGLU(a.hidden_size, spec.mlp["ff"], "gelu_tanh", dtype) if spec.mlp["kind"] == "dense" \
-                else SparseMoE(a.hidden_size, spec.mlp, dtype)
+                else (SparseGLU if a.expert_form == "glu" else SparseMoE)(a.hidden_size, spec.mlp, dtype)
 
     def new_state(self, *a):
         return self.mixer.new_state(*a)
 
     def forward(self, x, _residual, meta, cache=None):
-        h = self.input_layernorm(x, self.mlp.out_bias if self.mlp is not None else None)
+        if self.mlp_layernorm is not None:
+            h, hf = self.input_layernorm(x, self.mlp_layernorm)
+        else:
+            h = hf = self.input_layernorm(x, self.mlp.out_bias if self.mlp is not None else None)
         self.mixer(h, meta, cache, x)
         if self.mlp is not None:
-            self.mlp(h, x)
+            self.mlp(hf, x)
         return x, None
 
 
@@ -391,18 +430,26 @@ class Decoder(nn.Module):
     def __init__(self, a: HFArch, dtype):
         super().__init__()
         self.embed_tokens = nn.Embedding(a.vocab_size, a.hidden_size, dtype=dtype)
-        self.embedding_scale, self.hybrid = a.embedding_scale, a.layers is not None
+        self.embedding_scale, self.hybrid, self.bigram = a.embedding_scale, a.layers is not None, a.bigram
+        self.keeps_tokens = a.bigram is not None          # the state holds token ids: the embedding looks one back
+        if self.bigram is not None:
+            self.embed_pairs = nn.Embedding(self.bigram["buckets"] + 1, a.hidden_size, dtype=dtype)
         if self.hybrid:
             own = {i: ParallelLayer(a, a.layers[i], dtype) for i in {weight_owner(a.layers, i) for i in range(len(a.layers))}}
             # a layer with the weights of another one is the same module at two places, with a state at each
             self.layers = nn.ModuleList(own[weight_owner(a.layers, i)] for i in range(len(a.layers)))
-            self.norm = DynamicTanh(a.hidden_size, dtype)
+            self.norm = _block_norm(a, dtype)
         else:
             self.layers = nn.ModuleList(DecoderLayer(a, dtype) for _ in range(a.num_hidden_layers))
             self.norm = RMSNorm(a.hidden_size, a.rms_norm_eps, dtype)
 
-    def embed(self, ids):
-        """The residual stream the layers start from."""
+    def embed(self, ids, meta=None, tokens=None):
+        """The residual stream the layers start from.  ``meta`` and ``tokens`` (what the state keeps of earlier steps, or
+        None) matter where the embedding looks at the previous token."""
+        if self.bigram is not None:
+            return iops.embed_pairs(ids.reshape(-1), self.embed_tokens.weight, self.embed_pairs.weight, self.embedding_scale,
+                                    self.bigram["mul_prev"], self.bigram["mul_cur"], meta,
+                                    tokens.ids if tokens is not None else None)
         if self.hybrid:
             return iops.embed_scaled(ids.reshape(-1), self.embed_tokens.weight, self.embedding_scale)
         return self.embed_tokens(ids.reshape(-1))
@@ -482,8 +529,16 @@ class CausalLM(nn.Module):
         w = self.lm_head.weight
         return F.normalize(w.float(), dim=-1).to(w.dtype) if self.arch.norm_head else w
 
-    def hidden_states(self, input_ids, meta, caches=None, inputs_embeds=None):
-        x = inputs_embeds if inputs_embeds is not None else self.model.embed(input_ids)
+    def prepare_positions(self, length, device):
+        """Position tables for sequences of up to ``length`` tokens, made now rather than in a step."""
+        for m in self.modules():
+            if getattr(m, "rotary", None) is not None:
+                m.rotary.get(length, device)
+
+    def hidden_states(self, input_ids, meta, caches=None, inputs_embeds=None, tokens=None):
+        if inputs_embeds is not None and self.model.keeps_tokens:
+            raise NotImplementedError(f"{self.arch.family}: the embedding depends on token pairs, it takes ids only")
+        x = inputs_embeds if inputs_embeds is not None else self.model.embed(input_ids, meta, tokens)
         x = x.reshape(-1, x.shape[-1])
         if self.model.hybrid:
             iops.no_grad_check(x, self.lm_head.weight)
@@ -557,7 +612,7 @@ class CausalLM(nn.Module):
             parts = [torch.as_tensor(t, dtype=torch.long).reshape(-1) for t in tokens]
             counts, ids = [p.numel() for p in parts], torch.cat(parts).to(dev, non_blocking=True)
         meta = state.step_meta(slots, counts)
-        return self.hidden_states(ids, meta, state.layers, inputs_embeds=inputs_embeds), meta
+        return self.hidden_states(ids, meta, state.layers, inputs_embeds=inputs_embeds, tokens=state.tokens), meta
 
     @torch.no_grad()
     def logits(self, h):
@@ -591,6 +646,8 @@ class CausalLM(nn.Module):
         pre_emb = soft.get("embeds")
         n_kv = 0 if pre_kv is None else pre_kv.shape[2]
         n_emb = 0 if pre_emb is None else pre_emb.shape[0]
+        if (n_kv or n_emb) and self.model.keeps_tokens:
+            raise NotImplementedError(f"{a.family}: soft prefixes (the embedding depends on token pairs)")
         state = self.new_state(b, s + max_new_tokens + n_kv + n_emb)
         slots = [state.open() for _ in range(b)]
         if n_kv:

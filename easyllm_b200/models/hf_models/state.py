@@ -4,11 +4,13 @@
 gives it back; a slot that is used again starts from position 0, which every layer takes as "nothing before".  Each
 layer contributes one state object through ``layer.new_state``:
 
-* ``KVRows``: keys and values, ``[slots, capacity, kv_heads, dim]``, grown in whole blocks of positions;
+* ``PositionRows``: something for every position, ``[slots, capacity, ...]``, grown in whole blocks of positions; as
+  ``KVRows`` keys and values ``[.., kv_heads, dim]``, as ``LatentRows`` one latent and one rotated key part per position;
 * ``SlotTensors``: fixed-size tensors per slot (recurrent matrices, last inputs of a short convolution or a token shift);
 * a plain dict (the 8-bit cache of Qwen): dense batches of equal length only.
 
-``DecodeState.step_meta`` is the packed description of one step that the layers read.  All index tensors are built on
+What the embedding keeps (token ids by position, when it looks at the previous token) is one more ``PositionRows``,
+``DecodeState.tokens``.  ``DecodeState.step_meta`` is the packed description of one step that the layers read.  All index tensors are built on
 the host and copied once; ``DecodeGraph`` replays the one-token step of fixed slots as a CUDA graph, with the positions
 advanced on the device.
 """
@@ -19,17 +21,31 @@ import torch
 BLOCK = 256          # positions a key/value cache grows by
 
 
-class KVRows:
-    def __init__(self, slots, capacity, kv_heads, dim, vdim, device, dtype):
-        self.k = torch.zeros(slots, capacity, kv_heads, dim, dtype=dtype, device=device)
-        self.v = torch.zeros(slots, capacity, kv_heads, vdim, dtype=dtype, device=device)
+class PositionRows:
+    def __init__(self, slots, capacity, device, **shapes):
+        """``name=(shape, dtype)`` per tensor; each becomes an attribute ``[slots, capacity, *shape]``."""
+        self.names = list(shapes)
+        for name, (shape, dtype) in shapes.items():
+            setattr(self, name, torch.zeros(slots, capacity, *shape, dtype=dtype, device=device))
 
     def grow(self, slots, capacity):
-        for name in ("k", "v"):
+        for name in self.names:
             old = getattr(self, name)
             new = old.new_zeros(slots, capacity, *old.shape[2:])
             new[:old.shape[0], :old.shape[1]] = old
             setattr(self, name, new)
+
+
+class LatentRows(PositionRows):
+    """``c``: per position the normed latent followed by the rotated key part, rows padded to 8 elements."""
+
+    def __init__(self, slots, capacity, rank, rot, device, dtype):
+        super().__init__(slots, capacity, device, c=((-(-(rank + rot) // 8) * 8,), dtype))
+
+
+class KVRows(PositionRows):
+    def __init__(self, slots, capacity, kv_heads, dim, vdim, device, dtype):
+        super().__init__(slots, capacity, device, k=((kv_heads, dim), dtype), v=((kv_heads, vdim), dtype))
 
     def load_prefix(self, slots, k, v):
         """Fill positions ``0 .. n`` of ``slots`` with given keys / values ``[n, kv_heads, dim]`` (prefix tuning)."""
@@ -58,6 +74,8 @@ class DecodeState:
         self.device, self.dtype = device or w.device, dtype or w.dtype
         self.capacity = -(-capacity // BLOCK) * BLOCK
         self.layers = [layer.new_state(slots, self.capacity, self.device, self.dtype) for layer in model.model.layers]
+        self.tokens = PositionRows(slots, self.capacity, self.device, ids=((), torch.int32)) if model.model.keeps_tokens \
+            else None
         self.lengths = [0] * slots
         self.free = list(range(slots - 1, -1, -1))
 
@@ -90,6 +108,8 @@ class DecodeState:
             if not hasattr(st, "grow"):
                 raise ValueError("this cache cannot grow: it holds one dense batch of a fixed size")
             st.grow(slots, capacity)
+        if self.tokens is not None:
+            self.tokens.grow(slots, capacity)
         self.capacity = capacity
 
     # ---- one step ------------------------------------------------------------------------------
@@ -137,10 +157,11 @@ class DecodeGraph:
         # host-side bounds that hold for every replay
         self.meta.update(max_position=state.capacity, kv_bound=state.capacity, fresh=False, one_token=True)
         self.ids = torch.zeros(len(slots), dtype=torch.long, device=state.device)
+        model.prepare_positions(state.capacity, state.device)
         self.graph = torch.cuda.CUDAGraph()
         torch.cuda.synchronize()
         with torch.no_grad(), torch.cuda.graph(self.graph):
-            self.logits = model.logits(model.hidden_states(self.ids, self.meta, state.layers))
+            self.logits = model.logits(model.hidden_states(self.ids, self.meta, state.layers, tokens=state.tokens))
             for name in ("seq_pos0", "position_ids", "kv_len"):
                 self.meta[name].add_(1)
 

@@ -232,9 +232,23 @@ class RotaryTables:
             ntk = self.ntk_max_pos
             if ntk is not None and need <= ntk:
                 n = min(n, ntk) if n >= need else n
-            self.cos, self.sin = ref.rope_tables(self.head_dim, n, self.base, self.scale, device, ntk)
+            self.cos, self.sin = self._tables(n, device)
             self.cached = n
         return self.cos, self.sin
+
+    def _tables(self, n, device):
+        return ref.rope_tables(self.head_dim, n, self.base, self.scale, device, self.ntk_max_pos)
+
+
+class YarnRotaryTables(RotaryTables):
+    """Tables of ``ops.reference.yarn_frequencies``: per-pair frequency scaling, angles formed in double precision."""
+
+    def __init__(self, dims, base, scaling=None):
+        super().__init__(dims, base)
+        self.scaling = scaling
+
+    def _tables(self, n, device):
+        return ref.yarn_tables(self.head_dim, n, self.base, self.scaling, device)
 
 
 def alibi_slopes(n_heads):

@@ -8,6 +8,10 @@
 // scores, the softmax runs on the KT scores of a head per warp, and for the weighted sum a thread owns eight value
 // columns and a share of the tile's keys; the shares are added up once, at the end.  With more than one range per row a
 // second kernel merges the partial (max, sum, accumulator) triples; the sink joins the denominator at the end, once.
+// A window keeps the last `window` of a row's keys.  A gate multiplies head h's output of row t by sigmoid(gate[t][h]).
+//
+// Latent attention (one key row shared by all query heads, whose first dv columns are also the value, bf16) has a
+// kernel of its own, attn_latent_kernel: the products run on mma.sync m16n8k16 over a key tile that is read once.
 #include "vec.cuh"
 
 namespace ell {
@@ -22,7 +26,24 @@ struct AttnRowsArgs {
   const float *sink, *slopes;
   int n, H, G, d, dv, ldq, ldk, ldv, splits, range;
   float scale;
+  int window;                     // keys a row sees at most (INT_MAX: all)
+  const void* gate;               // [n, ldg] of the activation type, or null
+  int ldg;
 };
+
+// Keys row t sees: the last min(len, window) of its rows.
+struct RowKeys {
+  size_t base;
+  int len;
+};
+__device__ __forceinline__ RowKeys row_keys(const AttnRowsArgs& a, int t) {
+  const int all = a.len[t], len = min(all, a.window);
+  return {(size_t)a.base[t] + (all - len), len};
+}
+template <typename T>
+__device__ __forceinline__ float row_gate(const AttnRowsArgs& a, int t, int h) {
+  return a.gate == nullptr ? 1.f : sigmoid_f(to_f<T>(reinterpret_cast<const T*>(a.gate)[(size_t)t * a.ldg + h]));
+}
 
 // Shared memory: scaled queries [8][dp] | scores [8][KT] | statistics [8][4] | two stages of KT key rows, KT value rows.
 struct ArLayout {
@@ -56,8 +77,9 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
   float* p = qs + REP * dp;
   float* stat = p + REP * KT;                    // max, sum, rescale
   T* stages = reinterpret_cast<T*>(stat + REP * 4);
-  const int len = a.len[t];
-  const size_t base = a.base[t];
+  const RowKeys rk = row_keys(a, t);
+  const int len = rk.len;
+  const size_t base = rk.base;
   const int k0 = split * a.range, k1 = min(k0 + a.range, len);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // rows and columns the copies leave out must read as zero
@@ -236,7 +258,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
         f = expf(m - mm);
         den = l * f + expf(sk - mm);
       }
-      reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h0 + h) * a.dv + c] = from_f<T>(o * f / den);
+      reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h0 + h) * a.dv + c] = from_f<T>(o * f / den * row_gate<T>(a, t, h0 + h));
     } else {
       float* pt = a.part + (((size_t)t * a.H + h0 + h) * a.splits + split) * (a.dv + 2);
       if (c == 0) {
@@ -253,7 +275,8 @@ template <typename T>
 __global__ void __launch_bounds__(kArThreads) attn_rows_merge_kernel(const AttnRowsArgs a) {
   const int t = blockIdx.x, h = blockIdx.y;
   const float* pt = a.part + ((size_t)t * a.H + h) * a.splits * (a.dv + 2);
-  const int used = min(a.splits, (a.len[t] + a.range - 1) / a.range);
+  const int used = min(a.splits, (row_keys(a, t).len + a.range - 1) / a.range);
+  const float gate = row_gate<T>(a, t, h);
   float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
   for (int s = 0; s < used; ++s) m = fmaxf(m, pt[(size_t)s * (a.dv + 2)]);
   float den = a.sink != nullptr ? expf(a.sink[h] - m) : 0.f;
@@ -261,8 +284,257 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_merge_kernel(const AttnR
   for (int c = threadIdx.x; c < a.dv; c += kArThreads) {
     float o = 0.f;
     for (int s = 0; s < used; ++s) o = fmaf(pt[(size_t)s * (a.dv + 2) + 2 + c], expf(pt[(size_t)s * (a.dv + 2)] - m), o);
-    reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h) * a.dv + c] = from_f<T>(o / den);
+    reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h) * a.dv + c] = from_f<T>(o / den * gate);
   }
+}
+
+// ---- latent attention: all heads share one key row, its first dv columns are the value ---------------
+// A CTA of 8 warps takes (row t, 16 * MT query heads, a range of keys).  Tiles of 64 key rows come through two
+// shared-memory stages (cp.async); row strides are an odd number of 16-byte pieces, so ldmatrix meets no bank conflicts.
+//   scores   MT = 1: warp w multiplies keys 8 w .. 8 w + 7;  MT = 2: warps 0-3 take the first 16 heads, 4-7 the second,
+//            16 keys each.  Scores go to shared memory in fp32.
+//   softmax  a warp owns 2 * MT heads; two keys a lane; fp32 weights, their sum unrounded, the operand of P·V in bf16
+//   values   warp w owns columns [w, w + 1) * dv / 8 of all heads; the value operand is the key tile itself (ldmatrix
+//            with transposition); its rescaled accumulators stay in registers
+constexpr int kAlWarps = 8, kAlKeys = 64, kAlPStride = kAlKeys + 8, kAlSStride = kAlKeys + 4, kAlMaxNt = 8;
+
+__host__ __device__ inline int al_krow(int d) { return (d + 15) / 16 * 16 + 8; }
+static int al_bytes(int d, int MT) {
+  return (2 * kAlKeys + 16 * MT) * al_krow(d) * 2 + 16 * MT * (kAlPStride * 2 + kAlSStride * 4 + 16);
+}
+
+__device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <int MT>
+__global__ void __launch_bounds__(kAlWarps * 32) attn_latent_kernel(const AttnRowsArgs a) {
+  extern __shared__ __align__(16) uint8_t alsm[];
+  constexpr int HM = 16 * MT;
+  const int krow = al_krow(a.d), dp = krow - 8;
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(alsm);
+  __nv_bfloat16* kv = qs + HM * krow;
+  __nv_bfloat16* ps = kv + 2 * kAlKeys * krow;
+  float* ss = reinterpret_cast<float*>(ps + HM * kAlPStride);
+  float* stat = ss + HM * kAlSStride;                  // max | sum | rescale, HM each
+  const int t = blockIdx.x, h0 = blockIdx.y * HM, nh = min(HM, a.H - h0), split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const RowKeys rk = row_keys(a, t);
+  const int k0 = split * a.range, k1 = min(k0 + a.range, rk.len);
+  const __nv_bfloat16* kb = reinterpret_cast<const __nv_bfloat16*>(a.k) + rk.base * a.ldk;
+  const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(a.q) + (size_t)t * a.ldq + (size_t)h0 * a.d;
+  const int pieces = a.d / 8, padded = dp / 8;         // 16-byte pieces of a row
+  // rows and columns that the copies leave out read as zero
+  for (int i = threadIdx.x; i < HM * padded; i += kAlWarps * 32) {
+    const int h = i / padded, c = i % padded;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (h < nh && c < pieces) v = *reinterpret_cast<const uint4*>(qb + (size_t)h * a.d + c * 8);
+    *reinterpret_cast<uint4*>(qs + h * krow + c * 8) = v;
+  }
+  auto load_tile = [&](int kt, int buf) {
+    __nv_bfloat16* dst = kv + buf * kAlKeys * krow;
+    const int cnt = min(kAlKeys, k1 - kt);
+    for (int i = threadIdx.x; i < kAlKeys * padded; i += kAlWarps * 32) {
+      const int r = i / padded, c = i % padded;
+      if (r < cnt && c < pieces) cp_async16(dst + r * krow + c * 8, kb + (size_t)(kt + r) * a.ldk + c * 8);
+      else *reinterpret_cast<uint4*>(dst + r * krow + c * 8) = make_uint4(0, 0, 0, 0);
+    }
+    cp_async_commit();
+  };
+  if (threadIdx.x < HM) {
+    stat[threadIdx.x] = -INFINITY;
+    stat[HM + threadIdx.x] = 0.f;
+    stat[2 * HM + threadIdx.x] = 1.f;
+  }
+  const int nt = (a.dv / 8 + kAlWarps - 1) / kAlWarps;         // 8-column pieces of a warp
+  const int col0 = warp * nt * 8, mine = max(0, min(nt, (a.dv - col0) / 8));
+  float acc[MT][kAlMaxNt][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < kAlMaxNt; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+  const int g = lane >> 2, tq = lane & 3;
+  const int l8 = lane & 7, quad = lane >> 3;
+  if (k0 < k1) load_tile(k0, 0);
+  int buf = 0;
+  for (int kt = k0; kt < k1; kt += kAlKeys, buf ^= 1) {
+    if (kt + kAlKeys < k1) {
+      load_tile(kt + kAlKeys, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* ks = kv + buf * kAlKeys * krow;
+    // scores of 16 heads and MT * 8 keys
+    {
+      const int mt = MT == 1 ? 0 : warp >> 2, key0 = MT == 1 ? warp * 8 : (warp & 3) * 16;
+      float sc[MT][4];
+#pragma unroll
+      for (int n = 0; n < MT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) sc[n][i] = 0.f;
+      const __nv_bfloat16* qrow = qs + (mt * 16 + (quad & 1) * 8 + l8) * krow + (quad >> 1) * 8;
+      // 32 columns of 8 keys (MT 1), or 16 columns of 16 keys (MT 2), per ldmatrix
+      const __nv_bfloat16* krow_p = MT == 1 ? ks + (key0 + l8) * krow + quad * 8
+                                            : ks + (key0 + (quad >> 1) * 8 + l8) * krow + (quad & 1) * 8;
+      if (MT == 1) {
+        int c = 0;
+#pragma unroll 4
+        for (; c + 32 <= dp; c += 32) {
+          uint32_t a0[4], a1[4], b[4];
+          ldsm4(a0, qrow + c);
+          ldsm4(a1, qrow + c + 16);
+          ldsm4(b, krow_p + c);
+          mma_bf16(sc[0], a0, b[0], b[1]);
+          mma_bf16(sc[0], a1, b[2], b[3]);
+        }
+        if (c < dp) {                                    // a last single k-step: the lanes past it repeat its columns
+          uint32_t a0[4], b[4];
+          ldsm4(a0, qrow + c);
+          ldsm4(b, ks + (key0 + l8) * krow + c + (quad & 1) * 8);
+          mma_bf16(sc[0], a0, b[0], b[1]);
+        }
+      } else {
+#pragma unroll 4
+        for (int c = 0; c < dp; c += 16) {
+          uint32_t a0[4], b[4];
+          ldsm4(a0, qrow + c);
+          ldsm4(b, krow_p + c);
+          mma_bf16(sc[0], a0, b[0], b[1]);
+          mma_bf16(sc[MT - 1], a0, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < MT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int key = key0 + n * 8 + tq * 2 + (i & 1), hh = mt * 16 + g + (i >> 1) * 8;
+          ss[hh * kAlSStride + key] = kt + key < k1 ? sc[n][i] * a.scale : -INFINITY;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int x = 0; x < 2 * MT; ++x) {
+      const int hh = warp * 2 * MT + x;
+      const float s0 = ss[hh * kAlSStride + lane], s1 = ss[hh * kAlSStride + 32 + lane];
+      const float m_old = stat[hh], m = fmaxf(m_old, warp_max(fmaxf(s0, s1)));     // finite: the tile has a key
+      const float e0 = expf(s0 - m), e1 = expf(s1 - m);
+      ps[hh * kAlPStride + lane] = __float2bfloat16_rn(e0);
+      ps[hh * kAlPStride + 32 + lane] = __float2bfloat16_rn(e1);
+      const float sum = warp_sum(e0 + e1);
+      __syncwarp();
+      if (lane == 0) {
+        const float al = expf(m_old - m);
+        stat[hh] = m;
+        stat[HM + hh] = stat[HM + hh] * al + sum;
+        stat[2 * HM + hh] = al;
+      }
+    }
+    __syncthreads();
+    uint32_t pa[MT][kAlKeys / 16][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float r0 = stat[2 * HM + m * 16 + g], r1 = stat[2 * HM + m * 16 + g + 8];
+#pragma unroll
+      for (int n = 0; n < kAlMaxNt; ++n) {
+        acc[m][n][0] *= r0;
+        acc[m][n][1] *= r0;
+        acc[m][n][2] *= r1;
+        acc[m][n][3] *= r1;
+      }
+#pragma unroll
+      for (int k = 0; k < kAlKeys / 16; ++k)
+        ldsm4(pa[m][k], ps + (m * 16 + (quad & 1) * 8 + l8) * kAlPStride + k * 16 + (quad >> 1) * 8);
+    }
+#pragma unroll
+    for (int n = 0; n < kAlMaxNt; ++n) {
+      if (n < mine) {
+#pragma unroll
+        for (int k = 0; k < kAlKeys / 32; ++k) {         // 32 keys x 8 columns per ldmatrix
+          uint32_t b[4];
+          ldsm4_t(b, ks + (k * 32 + quad * 8 + l8) * krow + col0 + n * 8);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16(acc[m][n], pa[m][2 * k], b[0], b[1]);
+            mma_bf16(acc[m][n], pa[m][2 * k + 1], b[2], b[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int hh = m * 16 + g + r * 8;
+      if (hh >= nh) continue;
+      const size_t th = (size_t)t * a.H + h0 + hh;
+      const float l = stat[HM + hh];
+      if (a.splits == 1) {
+        const float f = row_gate<__nv_bfloat16>(a, t, h0 + hh) / l;
+        __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.out) + th * a.dv + col0 + tq * 2;
+#pragma unroll
+        for (int n = 0; n < kAlMaxNt; ++n)
+          if (n < mine)
+            *reinterpret_cast<__nv_bfloat162*>(o + n * 8) = __floats2bfloat162_rn(acc[m][n][2 * r] * f, acc[m][n][2 * r + 1] * f);
+      } else {
+        float* pt = a.part + (th * a.splits + split) * (a.dv + 2);
+        if (warp == 0 && tq == 0) {
+          pt[0] = stat[hh];
+          pt[1] = l;
+        }
+#pragma unroll
+        for (int n = 0; n < kAlMaxNt; ++n)
+          if (n < mine) *reinterpret_cast<float2*>(pt + 2 + col0 + n * 8 + tq * 2) = make_float2(acc[m][n][2 * r], acc[m][n][2 * r + 1]);
+      }
+    }
+}
+
+static int al_mt(int H) { return H > 16 ? 2 : 1; }
+
+// Ranges per row of the latent kernel: one CTA an SM, at least one tile each.
+static int attn_latent_splits(int n, int H, int max_len) {
+  const long long ctas = (long long)n * ((H + 16 * al_mt(H) - 1) / (16 * al_mt(H)));
+  long long s = kNumSMs / ctas;
+  const long long most = (max_len + kAlKeys - 1) / kAlKeys;
+  if (s > most) s = most;
+  if (s > 64) s = 64;
+  return s < 1 ? 1 : (int)s;
+}
+
+template <int MT>
+static int launch_attn_latent(const AttnRowsArgs& a, cudaStream_t stream) {
+  const int bytes = al_bytes(a.d, MT);
+  static int configured = 0;
+  if (bytes > configured) {
+    cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return (int)e;
+    configured = bytes;
+  }
+  attn_latent_kernel<MT><<<dim3(a.n, (a.H + 16 * MT - 1) / (16 * MT), a.splits), kAlWarps * 32, bytes, stream>>>(a);
+  if (a.splits > 1) attn_rows_merge_kernel<__nv_bfloat16><<<dim3(a.n, a.H), kArThreads, 0, stream>>>(a);
+  return launch_status();
+}
+
+// Shapes of the mma kernel; everything else runs on attn_rows_kernel.
+static bool attn_latent_fits(int d, int dv, int ldq, int ldk, int H) {
+  return d % 8 == 0 && dv % 8 == 0 && dv <= d && dv <= 8 * kAlWarps * kAlMaxNt && ldq % 8 == 0 && ldk % 8 == 0 &&
+         H <= 65535 && al_bytes(d, al_mt(H)) <= 227 * 1024;
 }
 
 // Query heads a CTA takes.
@@ -312,21 +584,52 @@ ELL_API long long ell_attn_rows_scratch(int n, int H, int G, int dv, int max_len
 }
 
 // Rows of ldq / ldk / ldv elements; max_len bounds len[] (it sets the number of ranges, longer rows would be cut).
+// window: keys a row sees (<= 0: all).  gate: rows of ldg elements of the activation type, or null.
 ELL_API int ell_attn_rows(const void* q, const void* k, const void* v, void* out, float* part, const int* base,
-                          const int* len, const float* sink, const float* slopes, int n, int H, int G, int d, int dv,
-                          int ldq, int ldk, int ldv, int max_len, float scale, int is_bf16, cudaStream_t stream) {
+                          const int* len, const float* sink, const float* slopes, const void* gate, int n, int H, int G,
+                          int d, int dv, int ldq, int ldk, int ldv, int ldg, int max_len, int window, float scale,
+                          int is_bf16, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (H % G || dv > 512 || d > 512 || H > 65535) return -2;
-  AttnRowsArgs a{q, k, v, out, part, base, len, sink, slopes, n, H, G, d, dv, ldq, ldk, ldv, 1, 0, scale};
+  if (H % G || dv > 8 * kArThreads || H > 65535) return -2;
+  if (window <= 0) window = 0x7fffffff;
+  if (max_len > window) max_len = window;
+  AttnRowsArgs a{q, k, v, out, part, base, len, sink, slopes, n, H, G, d, dv, ldq, ldk, ldv, 1, 0, scale, window, gate, ldg};
   a.splits = attn_rows_splits(n, H, G, max_len);
   a.range = ((max_len + a.splits - 1) / a.splits + 63) / 64 * 64;
   if (a.splits > 1 && part == nullptr) return -2;
   const int rep = H / G, per = ar_rep(rep);
   dim3 grid(n, G * ((rep + per - 1) / per), a.splits);
   const int esz = is_bf16 ? 2 : 4;
+  if (ar_layout(d, dv, esz, 16, per).bytes > 227 * 1024) return -2;
   const bool vec = (d * esz) % 16 == 0 && (dv * esz) % 16 == 0 && (ldk * esz) % 16 == 0 && (ldv * esz) % 16 == 0 &&
                    aligned_to(k, 16) && aligned_to(v, 16);
   if (is_bf16)
     return per == 4 ? launch_attn_rows<__nv_bfloat16, 4>(a, grid, vec, stream) : launch_attn_rows<__nv_bfloat16, 8>(a, grid, vec, stream);
   return per == 4 ? launch_attn_rows<float, 4>(a, grid, vec, stream) : launch_attn_rows<float, 8>(a, grid, vec, stream);
+}
+
+// Latent attention: q [n, H, d] (rows of ldq), one key row [d] per position (rows of ldk) whose first dv columns are the
+// value -> out [n, H, dv].  bf16 shapes the mma kernel takes run there, others on attn_rows.
+ELL_API long long ell_attn_latent_scratch(int n, int H, int d, int dv, int ldq, int ldk, int max_len, int window, int is_bf16) {
+  if (window > 0 && max_len > window) max_len = window;
+  if (!(is_bf16 && attn_latent_fits(d, dv, ldq, ldk, H))) return ell_attn_rows_scratch(n, H, 1, dv, max_len);
+  const int s = attn_latent_splits(n, H, max_len);
+  return s == 1 ? 0 : (long long)n * H * s * (dv + 2);
+}
+
+ELL_API int ell_attn_latent(const void* q, const void* k, void* out, float* part, const int* base, const int* len,
+                            const void* gate, int n, int H, int d, int dv, int ldq, int ldk, int ldg, int max_len, int window,
+                            float scale, int is_bf16, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(is_bf16 && attn_latent_fits(d, dv, ldq, ldk, H)))
+    return ell_attn_rows(q, k, k, out, part, base, len, nullptr, nullptr, gate, n, H, 1, d, dv, ldq, ldk, ldk, ldg, max_len,
+                         window, scale, is_bf16, stream);
+  if (!aligned_to(q, 16) || !aligned_to(k, 16) || !aligned_to(out, 16)) return -2;
+  if (window <= 0) window = 0x7fffffff;
+  if (max_len > window) max_len = window;
+  AttnRowsArgs a{q, k, k, out, part, base, len, nullptr, nullptr, n, H, 1, d, dv, ldq, ldk, ldk, 1, 0, scale, window, gate, ldg};
+  a.splits = attn_latent_splits(n, H, max_len);
+  a.range = ((max_len + a.splits - 1) / a.splits + kAlKeys - 1) / kAlKeys * kAlKeys;
+  if (a.splits > 1 && part == nullptr) return -2;
+  return al_mt(H) == 1 ? launch_attn_latent<1>(a, stream) : launch_attn_latent<2>(a, stream);
 }

@@ -312,6 +312,47 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         }
       }
       if (OUT == kOutBf16 || OUT == kOutBf16CE) {
+        if (FUSE == kFuseGroup && fuse.group_glu) {
+          // 64 accumulator columns are 32 gate and 32 up columns: two of them fill one box of 64 result columns
+          const float sc = fuse.row_scale[m0 + row_in_tile];
+#pragma unroll 1
+          for (int j = 0; j < BN / 64; ++j) {
+            uint8_t* buf = sC + (store_count & 1) * kEpiBufBytes;
+            if ((j & 1) == 0) {
+              if (leader) tma_store_wait_read<1>();
+              named_bar_sync(1, kEpiThreads);
+            }
+            uint32_t r[64];
+            tmem_ld_32x32(t_row + j * 64, r);
+            tmem_ld_32x32(t_row + j * 64 + 32, r + 32);
+            tmem_ld_wait();
+            uint8_t* row_ptr = buf + row_in_tile * 128;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+              uint32_t v[4];
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float g0 = __uint_as_float(r[c * 8 + 2 * e]), g1 = __uint_as_float(r[c * 8 + 2 * e + 1]);
+                const float u0 = __uint_as_float(r[32 + c * 8 + 2 * e]), u1 = __uint_as_float(r[32 + c * 8 + 2 * e + 1]);
+                const __nv_bfloat162 p = __floats2bfloat162_rn(__fdividef(g0, 1.f + __expf(-g0)) * u0 * sc,
+                                                               __fdividef(g1, 1.f + __expf(-g1)) * u1 * sc);
+                v[e] = *reinterpret_cast<const uint32_t*>(&p);
+              }
+              const int chunk = (j & 1) * 4 + c;
+              *reinterpret_cast<uint4*>(row_ptr + ((chunk ^ (row_in_tile & 7)) << 4)) = make_uint4(v[0], v[1], v[2], v[3]);
+            }
+            if (j & 1) {
+              fence_proxy_async_smem();
+              named_bar_sync(1, kEpiThreads);
+              if (leader) {
+                const int col = (n0 + (j - 1) * 64) / 2;
+                if (col < N / 2) tma_store_2d(&tmC, buf, col, m0);
+                tma_store_commit();
+              }
+              ++store_count;
+            }
+          }
+        } else
 #pragma unroll 1
         for (int j = 0; j < u.bn / 64; ++j) {
           uint8_t* buf = sC + (store_count & 1) * kEpiBufBytes;
@@ -527,14 +568,16 @@ static int make_tmap_2d(CUtensorMap* map, CUtensorMapDataType dt, const void* pt
   return r == CUDA_SUCCESS ? 0 : -12;
 }
 
-// 3-D bf16 tensor map over [rows, heads, dim] (dim contiguous, heads packed): boxes of one head, zero-filled past `dim`.
+// 3-D bf16 tensor map over [rows, heads, dim] (dim contiguous; heads packed, or head_stride_bytes apart): boxes of one
+// head, zero-filled past `dim`.
 int make_tmap_bf16_heads(CUtensorMap* map, const void* ptr, uint64_t dim, uint64_t heads, uint64_t rows,
-                         uint64_t row_stride_bytes, uint32_t box_dim, uint32_t box_rows) {
+                         uint64_t row_stride_bytes, uint32_t box_dim, uint32_t box_rows, uint64_t head_stride_bytes) {
   EncodeTiledFn fn = get_encode_fn();
   if (!fn) return -10;
-  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (row_stride_bytes & 15) || ((dim * 2) & 15)) return -11;
+  if (head_stride_bytes == 0) head_stride_bytes = dim * 2;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (row_stride_bytes & 15) || (head_stride_bytes & 15)) return -11;
   cuuint64_t dims[3] = {dim, heads, rows};
-  cuuint64_t strides[2] = {dim * 2, row_stride_bytes};
+  cuuint64_t strides[2] = {head_stride_bytes, row_stride_bytes};
   cuuint32_t box[3] = {box_dim, 1, box_rows};
   cuuint32_t estr[3] = {1, 1, 1};
   CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
@@ -704,19 +747,24 @@ ELL_API int ell_gemm_bf16(const void* A, const void* B, void* C, const void* bia
 // Grouped product for rows sorted by expert: C[rows, N] (bf16) = A[rows, K] · W[expert of the row tile][N, K]^T, where
 // every expert's rows start at a multiple of 128.  W is [experts * N, K]; `rows` is the capacity of A and C (a multiple
 // of 128), *n_row_tiles the 128-row tiles in use.  row_scale (fp32 [rows] or null): C = (row_scale relu(.))^2.
+// glu: an expert's N rows alternate in blocks of 32 gate and 32 up rows, C [rows, N / 2] = row_scale silu(gate) up.
 ELL_API int ell_gemm_grouped(const void* A, const void* W, void* C, const int* tile_expert, const int* n_row_tiles,
-                             const float* row_scale, int rows, int N, int K, int experts, int* err, cudaStream_t stream) {
+                             const float* row_scale, int rows, int N, int K, int experts, int glu, int* err,
+                             cudaStream_t stream) {
   if (rows <= 0 || N <= 0 || K <= 0) return 0;
   if (rows % kBM || N % 8 || K % 8) return -2;
+  if (glu && (N % 64 || row_scale == nullptr)) return -2;
   const int BN = N > 128 ? 256 : 128;
   CUtensorMap tA, tB, tC;
   int rc = make_tmap_bf16_2d(&tA, A, (uint64_t)K, (uint64_t)rows, (uint64_t)K * 2, kBK, kBM);
   if (rc) return rc;
   rc = make_tmap_bf16_2d(&tB, W, (uint64_t)K, (uint64_t)experts * N, (uint64_t)K * 2, kBK, BN);
   if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tC, C, (uint64_t)N, (uint64_t)rows, (uint64_t)N * 2, 64, 128);
+  const uint64_t cols = glu ? N / 2 : N;
+  rc = make_tmap_bf16_2d(&tC, C, cols, (uint64_t)rows, cols * 2, 64, 128);
   if (rc) return rc;
   FuseArgs f{};
+  f.group_glu = glu;
   f.tile_expert = tile_expert;
   f.n_row_tiles = n_row_tiles;
   f.row_scale = row_scale;

@@ -20,7 +20,8 @@
 //            full-size output.  Two-shot: each byte crosses NVLink once per phase.
 //  kFuseGroup  no collective: a grouped product for rows sorted by expert.  Row tile i multiplies the weight rows of
 //            expert tile_expert[i] of a stacked [experts * N, K] operand; the number of row tiles is read on the device.
-//            With row_scale the epilogue writes (row_scale relu(c))^2.
+//            With row_scale the epilogue writes (row_scale relu(c))^2, or, for gated experts (group_glu), whose weight
+//            rows alternate in blocks of 32 gate and 32 up rows, row_scale silu(gate) up in N / 2 columns.
 // Flags are epoch counters that only grow; a per-peer `done` word tells a producer that the consumer has
 // finished the previous epoch before a buffer is overwritten.  Every wait is bounded and reports through the
 // error word.  Tensor maps only ever cover this GPU's memory and no load names more than one destination CTA.
@@ -72,7 +73,8 @@ struct FuseArgs {
   unsigned long long data_bytes;         // size of each data_ptrs[] buffer: every computed offset is checked against it
   const int* tile_expert;                // Group: expert of every row tile
   const int* n_row_tiles;                // Group: number of row tiles in use
-  const float* row_scale;                // Group: per-row scale of the squared-relu epilogue, or null
+  const float* row_scale;                // Group: per-row scale of the activation in the epilogue, or null
+  int group_glu;                         // Group: the activation is silu(gate) * up over interleaved columns
   int rs_lag_q;                          // CTA-pair reduce-scatter: own tiles trail the peers' by this many quarter waves (0: default)
 };
 

@@ -1,5 +1,6 @@
-// Elementwise and short-reduction kernels of the hybrid decoder layers (inference): scaled embedding into the fp32
-// stream, the dynamic-tanh norm, gated activations, token shift, head norm with gate, key/value cache writes.
+// Elementwise and short-reduction kernels of the hybrid decoder layers (inference): scaled embedding (with a table of
+// token pairs) into the fp32 stream, the dynamic-tanh norm, layer norms that share their statistics, gated activations,
+// token shift, head norm with gate, key/value cache writes, the rotations and the norm of latent attention.
 //
 // Templated on the activation type (bf16 for serving, fp32 for exact runs); every value is computed in fp32.  Compiled
 // without fast-math: tanh, exp and the divisions are the accurate ones, the fp32 runs depend on them.
@@ -241,6 +242,187 @@ __global__ void kv_append_kernel(const T* __restrict__ k, const T* __restrict__ 
   }
 }
 
+// out[t] = table[id] * scale + pairs[(previous id * mul_prev + id * mul_cur) mod buckets]; a sequence's first token takes
+// row `buckets`.  One CTA per token.  The previous token is the row before, or, for the first row of a sequence that goes
+// on, the entry before this one's in `hist` (token ids by position: row base[t] + len[t] - 1 is this token's, and is
+// written).  hist null: every sequence starts in this batch.
+template <typename T, int V>
+__global__ void embed_pairs_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
+                                   const T* __restrict__ pairs, float* __restrict__ out, const int* __restrict__ row_start,
+                                   const int* __restrict__ base, const int* __restrict__ len, int* __restrict__ hist, int W,
+                                   long long rows, long long buckets, long long mul_prev, long long mul_cur, float scale,
+                                   int* __restrict__ err) {
+  const int t = blockIdx.x;
+  const long long id = ids[t];
+  const bool first_row = row_start[t] == t;
+  const int place = hist != nullptr ? len[t] - 1 : 0;
+  const size_t entry = hist != nullptr ? (size_t)base[t] + place : 0;
+  long long prev = -1;
+  if (!first_row) prev = ids[t - 1];
+  else if (place > 0) prev = hist[entry - 1];
+  const bool bad = id < 0 || id >= rows || prev >= rows;
+  if (bad && threadIdx.x == 0) atomicCAS(err, 0, 31);
+  const long long row = bad ? 0 : (prev < 0 ? buckets : (prev * mul_prev + id * mul_cur) % buckets);
+  const T* a = table + (bad ? 0 : id) * W;
+  const T* b = pairs + row * W;
+  for (int c = threadIdx.x * V; c < W; c += blockDim.x * V) {
+    float f[V], g[V];
+    load_v<V>(a + c, f);
+    load_v<V>(b + c, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) f[j] = bad ? 0.f : fmaf(f[j], scale, g[j]);
+    store_v<V>(out + (size_t)t * W + c, f);
+  }
+  if (hist != nullptr && threadIdx.x == 0) hist[entry] = bad ? 0 : (int)id;
+}
+
+// Layer norms without a bias of one fp32 row, with one or two weights: y_i = (x - mean) / sqrt(variance + eps) * w_i.  One
+// CTA per row; IT pieces of 4 columns a thread stay in registers (IT = 0: any width, re-read).
+constexpr int kLnPairThreads = 256;
+
+__device__ __forceinline__ float ln_block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < kLnPairThreads / 32; ++i) s += red[i];
+  return s;
+}
+
+template <typename T, int IT>
+__global__ void __launch_bounds__(kLnPairThreads)
+layer_norms_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                   T* __restrict__ y1, T* __restrict__ y2, int W, float eps) {
+  __shared__ float red[2][kLnPairThreads / 32];
+  const float* row = x + (size_t)blockIdx.x * W;
+  T* o1 = y1 + (size_t)blockIdx.x * W;
+  T* o2 = y2 + (size_t)blockIdx.x * W;
+  if (IT > 0) {
+    float f[IT > 0 ? IT : 1][4];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int c = (i * kLnPairThreads + threadIdx.x) * 4;
+      if (c < W) load_v<4>(row + c, f[i]);
+      else f[i][0] = f[i][1] = f[i][2] = f[i][3] = 0.f;
+      s += (f[i][0] + f[i][1]) + (f[i][2] + f[i][3]);
+    }
+    const float mean = ln_block_sum(s, red[0]) / W;
+    float q = 0.f;
+#pragma unroll
+    for (int i = 0; i < IT; ++i)
+      if ((i * kLnPairThreads + threadIdx.x) * 4 < W)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          f[i][j] -= mean;
+          q = fmaf(f[i][j], f[i][j], q);
+        }
+    const float r = 1.f / sqrtf(ln_block_sum(q, red[1]) / W + eps);
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int c = (i * kLnPairThreads + threadIdx.x) * 4;
+      if (c < W) {
+        float w[4], o[4];
+        load_v<4>(w1 + c, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = f[i][j] * r * w[j];
+        store_v<4>(o1 + c, o);
+        if (w2 != nullptr) {
+          load_v<4>(w2 + c, w);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) o[j] = f[i][j] * r * w[j];
+          store_v<4>(o2 + c, o);
+        }
+      }
+    }
+  } else {
+    float s = 0.f;
+    for (int c = threadIdx.x; c < W; c += kLnPairThreads) s += row[c];
+    const float mean = ln_block_sum(s, red[0]) / W;
+    float q = 0.f;
+    for (int c = threadIdx.x; c < W; c += kLnPairThreads) q = fmaf(row[c] - mean, row[c] - mean, q);
+    const float r = 1.f / sqrtf(ln_block_sum(q, red[1]) / W + eps);
+    for (int c = threadIdx.x; c < W; c += kLnPairThreads) {
+      const float v = (row[c] - mean) * r;
+      o1[c] = from_f<T>(v * w1[c]);
+      if (w2 != nullptr) o2[c] = from_f<T>(v * w2[c]);
+    }
+  }
+}
+
+// Latent attention between its input and its score products, in place on the projection rows z [n, ldz], whose columns
+// are H queries of [dim unrotated, rot rotated], the latent of `rank`, one rotated key part:
+//   rotated query parts -> z, or, with q_dst, to q_dst [n, H, q_stride]: neighbouring dimensions 2i, 2i+1 are a pair,
+//     turned by the angle tables cos / sin [position, pairs]; dimensions past 2 * pairs pass unchanged
+//   latent -> divided by its root mean square, times norm_w;  key part -> rotated
+// Latent and key part also go to cache row base[t] + len[t] - 1 (rows of ldc), if there is a cache.  One CTA per token.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+latent_inputs_kernel(T* __restrict__ z, T* __restrict__ q_dst, T* __restrict__ cache, const float* __restrict__ norm_w,
+                     const float* __restrict__ cosT, const float* __restrict__ sinT, const int* __restrict__ pos,
+                     const int* __restrict__ base, const int* __restrict__ len, int H, int dim, int rot, int rank, int pairs,
+                     int ldz, int q_stride, int ldc, float eps) {
+  __shared__ float red[8];
+  const int t = blockIdx.x;
+  constexpr int VL = V == 8 ? 8 : 1;                    // pieces of the latent (any rank)
+  T* row = z + (size_t)t * ldz;
+  const float* ct = cosT + (size_t)pos[t] * pairs;
+  const float* st = sinT + (size_t)pos[t] * pairs;
+  auto turn = [&](const T* src, T* dst, int c) {        // V consecutive dimensions from c on (V even)
+    float f[V];
+    load_v<V>(src + c, f);
+#pragma unroll
+    for (int j = 0; j < V / 2; ++j) {
+      const int i = c / 2 + j;
+      if (i < pairs) {
+        const float u = f[2 * j], v = f[2 * j + 1], cs = ct[i], sn = st[i];
+        f[2 * j] = u * cs - v * sn;
+        f[2 * j + 1] = v * cs + u * sn;
+      }
+    }
+    store_v<V>(dst + c, f);
+  };
+  const int per = rot / V, qw = dim + rot;
+  for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+    const int h = i / per, c = (i % per) * V;
+    const T* src = row + (size_t)h * qw + dim;
+    turn(src, q_dst != nullptr ? q_dst + ((size_t)t * H + h) * q_stride : row + (size_t)h * qw + dim, c);
+  }
+  T* lat = row + (size_t)H * qw;
+  T* crow = cache != nullptr ? cache + ((size_t)base[t] + len[t] - 1) * ldc : nullptr;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VL; c < rank; c += blockDim.x * VL) {
+    float f[VL];
+    load_v<VL>(lat + c, f);
+#pragma unroll
+    for (int j = 0; j < VL; ++j) ss = fmaf(f[j], f[j], ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) ss += red[i];
+  const float r = 1.f / sqrtf(ss / rank + eps);
+  for (int c = threadIdx.x * VL; c < rank; c += blockDim.x * VL) {
+    float f[VL], w[VL];
+    load_v<VL>(lat + c, f);
+    load_v<VL>(norm_w + c, w);
+#pragma unroll
+    for (int j = 0; j < VL; ++j) f[j] = f[j] * r * w[j];
+    store_v<VL>(lat + c, f);
+    if (crow != nullptr) store_v<VL>(crow + c, f);
+  }
+  T* kr = lat + rank;
+  for (int c = threadIdx.x * V; c < rot; c += blockDim.x * V) {
+    turn(kr, kr, c);
+    if (crow != nullptr) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) crow[rank + c + j] = kr[c + j];
+    }
+  }
+}
+
 }  // namespace ell
 
 using namespace ell;
@@ -342,5 +524,63 @@ ELL_API int ell_kv_append(const void* k, const void* v_, void* kc, void* vc, con
                  aligned_to(kc, 16) && aligned_to(vc, 16);
   const int g = grid_for((long long)n * ((dk + dv) / (v ? 4 : 1)), 256);
   ELL_TV(v, kv_append_kernel, g, 256, (const T*)k, (const T*)v_, (T*)kc, (T*)vc, base, len, n, dk, dv, ldk, ldv);
+  return launch_status();
+}
+
+// hist (and base / len): token ids by position, or null.
+ELL_API int ell_embed_pairs(const long long* ids, const void* table, const void* pairs, float* out, const int* row_start,
+                            const int* base, const int* len, int* hist, int n, int W, long long rows, long long buckets,
+                            long long mul_prev, long long mul_cur, float scale, int is_bf16, int* err, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (buckets <= 0 || mul_prev < 0 || mul_cur < 0) return -2;
+  const bool v = W % 4 == 0 && aligned_to(table, 16) && aligned_to(pairs, 16) && aligned_to(out, 16);
+  ELL_TV(v, embed_pairs_kernel, n, 256, ids, (const T*)table, (const T*)pairs, out, row_start, base, len, hist, W, rows,
+         buckets, mul_prev, mul_cur, scale, err);
+  return launch_status();
+}
+
+// y1 = norm(x) w1, and with w2 also y2 = norm(x) w2.
+ELL_API int ell_layer_norms(const float* x, const float* w1, const float* w2, void* y1, void* y2, int n, int W, float eps,
+                            int is_bf16, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const bool v = W % 4 == 0 && W <= 8 * 4 * kLnPairThreads && aligned_to(x, 16) && aligned_to(w1, 16) &&
+                 aligned_to(w2, 16) && aligned_to(y1, 16) && aligned_to(y2, 16);
+  const int it = !v ? 0 : (W + 4 * kLnPairThreads - 1) / (4 * kLnPairThreads);
+#define ELL_LN(IT)                                                                                                     \
+  do {                                                                                                                 \
+    if (is_bf16)                                                                                                       \
+      layer_norms_kernel<__nv_bfloat16, IT><<<n, kLnPairThreads, 0, stream>>>(x, w1, w2, (__nv_bfloat16*)y1,           \
+                                                                             (__nv_bfloat16*)y2, W, eps);             \
+    else                                                                                                               \
+      layer_norms_kernel<float, IT><<<n, kLnPairThreads, 0, stream>>>(x, w1, w2, (float*)y1, (float*)y2, W, eps);      \
+  } while (0)
+  if (it == 0) ELL_LN(0);
+  else if (it == 1) ELL_LN(1);
+  else if (it == 2) ELL_LN(2);
+  else if (it <= 4) ELL_LN(4);
+  else ELL_LN(8);
+#undef ELL_LN
+  return launch_status();
+}
+
+// q_dst null: queries are rotated in place.  cache null: nothing is kept.  rot is even.
+ELL_API int ell_latent_inputs(void* z, void* q_dst, void* cache, const float* norm_w, const float* cosT, const float* sinT,
+                              const int* pos, const int* base, const int* len, int n, int H, int dim, int rot, int rank,
+                              int pairs, int ldz, int q_stride, int ldc, float eps, int is_bf16, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (rot % 2 || 2 * pairs > rot || rank < 1) return -2;
+  const bool v = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && ldz % 8 == 0 && q_stride % 8 == 0 && ldc % 8 == 0 &&
+                 aligned_to(z, 16) && aligned_to(q_dst, 16) && aligned_to(cache, 16) && aligned_to(norm_w, 16);
+#define ELL_LAT(T, V)                                                                                                   \
+  latent_inputs_kernel<T, V><<<n, 256, 0, stream>>>((T*)z, (T*)q_dst, (T*)cache, norm_w, cosT, sinT, pos, base, len, H, \
+                                                    dim, rot, rank, pairs, ldz, q_stride, ldc, eps)
+  if (is_bf16) {
+    if (v) ELL_LAT(__nv_bfloat16, 8);
+    else ELL_LAT(__nv_bfloat16, 2);
+  } else {
+    if (v) ELL_LAT(float, 8);
+    else ELL_LAT(float, 2);
+  }
+#undef ELL_LAT
   return launch_status();
 }

@@ -91,20 +91,21 @@ __device__ __forceinline__ void mma_16816(float* c, uint32_t a0, uint32_t a1, ui
       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// MT tiles of 8 rows of x.  Rows of W and of x past the end are clamped (their results are dropped); k past the end is
+// MT tiles of 8 rows of x (from row blockIdx.y * 8 MT on).  Rows of W and of x past the end are clamped (their results are dropped); k past the end is
 // clamped too, with x taken as zero.
 template <int MT>
 __global__ void __launch_bounds__(kMvWarps * 32) matvec_mma_kernel(const MatvecArgs a) {
   __shared__ float red[kMvWarps][16][8 * MT + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int ks = a.ks, part = warp % ks, n0 = (blockIdx.x * (kMvWarps / ks) + warp / ks) * 16;
-  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + blockIdx.z * a.xb;
+  const int m0 = blockIdx.y * 8 * MT, M = a.M - m0;
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + blockIdx.z * a.xb + (size_t)m0 * a.ldx;
   const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.w) + blockIdx.z * a.wb;
   const __nv_bfloat16* w0 = w + (size_t)min(n0 + g, a.N - 1) * a.K;
   const __nv_bfloat16* w1 = w + (size_t)min(n0 + g + 8, a.N - 1) * a.K;
   const __nv_bfloat16* xr[MT];
 #pragma unroll
-  for (int m = 0; m < MT; ++m) xr[m] = x + (size_t)min(m * 8 + g, a.M - 1) * a.ldx;
+  for (int m = 0; m < MT; ++m) xr[m] = x + (size_t)min(m * 8 + g, M - 1) * a.ldx;
   float c0[MT][4], c1[MT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -146,12 +147,12 @@ __global__ void __launch_bounds__(kMvWarps * 32) matvec_mma_kernel(const MatvecA
   const int rows = (kMvWarps / ks) * 16;
   for (int e = threadIdx.x; e < rows * 8 * MT; e += kMvWarps * 32) {
     const int r = e % rows, m = e / rows, n = blockIdx.x * rows + r;
-    if (n >= a.N || m >= a.M) continue;
+    if (n >= a.N || m >= M) continue;
     float v = 0.f;
     for (int p = 0; p < ks; ++p) v += red[(r >> 4) * ks + p][r & 15][m];
     if (a.bias != nullptr) v += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.bias)[n]);
     if (a.act_tanh) v = tanhf(v);
-    const size_t o = blockIdx.z * a.ob + (size_t)m * a.ldo + n;
+    const size_t o = blockIdx.z * a.ob + (size_t)(m0 + m) * a.ldo + n;
     if (a.accumulate) reinterpret_cast<float*>(a.out)[o] += v;
     else if (a.out_f32) reinterpret_cast<float*>(a.out)[o] = v;
     else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16_rn(v);
@@ -161,9 +162,10 @@ __global__ void __launch_bounds__(kMvWarps * 32) matvec_mma_kernel(const MatvecA
 static int launch_matvec_mma(MatvecArgs a, int batch, cudaStream_t stream) {
   const int nkb = (a.K + 31) / 32, tiles = (a.N + 15) / 16;
   a.ks = kMvWarps;
-  while (a.ks > 1 && (nkb < 4 * a.ks || (long long)tiles * batch * a.ks > 64LL * kNumSMs)) a.ks /= 2;
+  while (a.ks > 1 && (nkb < 4 * a.ks || (long long)tiles * batch * ((a.M + 15) / 16) * a.ks > 64LL * kNumSMs)) a.ks /= 2;
   const int per = kMvWarps / a.ks;
-  dim3 grid((tiles + per - 1) / per, 1, batch);
+  dim3 grid((tiles + per - 1) / per, (a.M + 15) / 16, batch);
+  if (grid.y > 65535) return -2;
   if (a.M <= 8) matvec_mma_kernel<1><<<grid, kMvWarps * 32, 0, stream>>>(a);
   else matvec_mma_kernel<2><<<grid, kMvWarps * 32, 0, stream>>>(a);
   return launch_status();
@@ -191,19 +193,21 @@ int dispatch_matvec(const MatvecArgs& a, int batch, bool vec, cudaStream_t strea
 }
 
 // ---- mixture of experts: routing, and the per-token products of a few tokens -----------------------
-// One warp per token: the `top` largest router logits (ties: the lower index), scores sigmoid(z).
-__global__ void moe_route_kernel(const float* __restrict__ z, int* __restrict__ idx, float* __restrict__ w, int n, int E,
-                                 int top, int ldz) {
+// One warp per token: the `top` largest router logits (ties: the lower index); scores sigmoid(z), or the softmax over the
+// chosen logits.  bias [E] (or null) is added to the logits first.
+__global__ void moe_route_kernel(const float* __restrict__ z, const float* __restrict__ bias, int* __restrict__ idx,
+                                 float* __restrict__ w, int n, int E, int top, int ldz, int softmax) {
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (t >= n) return;
   const float* row = z + (size_t)t * ldz;
   uint32_t taken = 0;                                  // bit i: expert 32 i + lane
+  float largest = 0.f, sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int be = 0x7fffffff;
     for (int i = 0; 32 * i + lane < E; ++i)
       if (!(taken >> i & 1)) {
-        const float v = row[32 * i + lane];
+        const float v = row[32 * i + lane] + (bias != nullptr ? bias[32 * i + lane] : 0.f);
         if (v > best || be == 0x7fffffff) {
           best = v;
           be = 32 * i + lane;
@@ -220,23 +224,33 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int* __restrict__ 
     }
     if ((be & 31) == lane) taken |= 1u << (be >> 5);
     if (lane == 0) {
+      if (k == 0) largest = best;
+      const float e = softmax ? expf(best - largest) : sigmoid_f(best);
+      sum += e;
       idx[t * top + k] = be;
-      w[t * top + k] = sigmoid_f(best);
+      w[t * top + k] = e;
     }
   }
+  if (softmax && lane == 0)
+    for (int k = 0; k < top; ++k) w[t * top + k] /= sum;
 }
 
-// hid[slot][f] = (w_slot relu(up_e[f] . h_token))^2 for slot = token * top + k; a warp computes two hidden units.
-template <typename T, bool VEC>
+// For slot = token * top + k, a warp multiplies two weight rows of expert e = idx[slot] with the token:
+//   GLU false  hidden units f0, f0 + 1 of up [E, F, W]:  hid[slot][f] = (w_slot relu(up_e[f] . h))^2
+//   GLU true   the gate and up rows of one hidden unit of [E, 2 F, W], which alternate in blocks of `block` rows:
+//              hid[slot][f] = w_slot silu(gate_e[f] . h) (up_e[f] . h)
+template <typename T, bool VEC, bool GLU>
 __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, const T* __restrict__ up,
                                                      const int* __restrict__ idx, const float* __restrict__ wgt,
-                                                     T* __restrict__ hid, int top, int F, int W) {
+                                                     T* __restrict__ hid, int top, int F, int W, int block) {
   const int slot = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int f0 = (blockIdx.x * 8 + warp) * 2;
+  const int f0 = (blockIdx.x * 8 + warp) * (GLU ? 1 : 2);
   if (f0 >= F) return;
   const T* x = h + (size_t)(slot / top) * W;
-  const T* u0 = up + ((size_t)idx[slot] * F + f0) * W;
-  const bool two = f0 + 1 < F;
+  const T* u0 = GLU ? up + ((size_t)idx[slot] * 2 * F + (size_t)(f0 / block) * 2 * block + f0 % block) * W
+                    : up + ((size_t)idx[slot] * F + f0) * W;
+  const bool two = GLU || f0 + 1 < F;
+  const size_t second = GLU ? (size_t)block * W : (two ? W : 0);
   float a0 = 0.f, a1 = 0.f;
 #pragma unroll 2
   for (int k = lane * 8; k < W; k += 256) {
@@ -244,14 +258,14 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, co
     if (VEC) {
       load_v<8>(x + k, xf);
       load_v<8>(u0 + k, w0);
-      load_v<8>(u0 + (two ? W : 0) + k, w1);
+      load_v<8>(u0 + second + k, w1);
     } else {
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const bool in = k + j < W;
         xf[j] = in ? to_f<T>(x[k + j]) : 0.f;
         w0[j] = in ? to_f<T>(u0[k + j]) : 0.f;
-        w1[j] = in ? to_f<T>(u0[(two ? W : 0) + k + j]) : 0.f;
+        w1[j] = in ? to_f<T>(u0[second + k + j]) : 0.f;
       }
     }
 #pragma unroll
@@ -264,6 +278,10 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, co
   a1 = warp_sum(a1);
   if (lane == 0) {
     const float s = wgt[slot];
+    if (GLU) {
+      hid[(size_t)slot * F + f0] = from_f<T>(s * silu_f(a0) * a1);
+      return;
+    }
     a0 = s * fmaxf(a0, 0.f);
     a1 = s * fmaxf(a1, 0.f);
     hid[(size_t)slot * F + f0] = from_f<T>(a0 * a0);
@@ -396,26 +414,30 @@ ELL_API int ell_matvec(const void* x, const void* w, const void* bias, void* out
   const int esz = is_bf16 ? 2 : 4;
   const bool vec = K % 8 == 0 && (ldx * esz) % 16 == 0 && aligned_to(x, 16) && aligned_to(w, 16) && (xb * esz) % 16 == 0 &&
                    (wb * esz) % 16 == 0;
-  if (is_bf16 && vec && M <= 16) return launch_matvec_mma(a, batch, stream);
+  if (is_bf16 && vec) return launch_matvec_mma(a, batch, stream);
   return is_bf16 ? dispatch_matvec<__nv_bfloat16>(a, batch, vec, stream) : dispatch_matvec<float>(a, batch, vec, stream);
 }
 
-ELL_API int ell_moe_route(const float* z, int* idx, float* w, int n, int E, int top, int ldz, cudaStream_t stream) {
+ELL_API int ell_moe_route(const float* z, const float* bias, int* idx, float* w, int n, int E, int top, int ldz, int softmax,
+                          cudaStream_t stream) {
   if (n <= 0) return 0;
   if (E > 1024 || top > E || top < 1) return -2;
-  moe_route_kernel<<<(n + 7) / 8, 256, 0, stream>>>(z, idx, w, n, E, top, ldz);
+  moe_route_kernel<<<(n + 7) / 8, 256, 0, stream>>>(z, bias, idx, w, n, E, top, ldz, softmax);
   return launch_status();
 }
 
 // acc [n, W] fp32 += experts; up [E, F, W], down [E, W, F]; hid: scratch [n * top, F] of the activation type.
+// glu_block > 0: gated experts, up [E, 2 F, W] with gate and up rows in alternating blocks of glu_block (a divisor of F).
 ELL_API int ell_moe_rows(const void* h, const void* up, const void* down, const int* idx, const float* w, void* hid,
-                         float* acc, int n, int top, int F, int W, int is_bf16, cudaStream_t stream) {
+                         float* acc, int n, int top, int F, int W, int glu_block, int is_bf16, cudaStream_t stream) {
   if (n <= 0) return 0;
   if ((long long)n * top > 65535) return -2;
   const bool v = F % 8 == 0 && W % 8 == 0 && aligned_to(h, 16) && aligned_to(up, 16) && aligned_to(down, 16) && aligned_to(hid, 16);
-  dim3 gu((F + 15) / 16, n * top), gd((W + 15) / 16, n);
+  if (glu_block < 0 || (glu_block > 0 && F % glu_block)) return -2;
+  dim3 gu(glu_block ? (F + 7) / 8 : (F + 15) / 16, n * top), gd((W + 15) / 16, n);
 #define ELL_MOE_ROWS(T, V)                                                                                          \
-  moe_up_kernel<T, V><<<gu, 256, 0, stream>>>((const T*)h, (const T*)up, idx, w, (T*)hid, top, F, W);               \
+  if (glu_block) moe_up_kernel<T, V, true><<<gu, 256, 0, stream>>>((const T*)h, (const T*)up, idx, w, (T*)hid, top, F, W, glu_block); \
+  else moe_up_kernel<T, V, false><<<gu, 256, 0, stream>>>((const T*)h, (const T*)up, idx, w, (T*)hid, top, F, W, 1); \
   moe_down_kernel<T, V><<<gd, 256, 0, stream>>>((const T*)hid, (const T*)down, idx, acc, top, F, W);
   if (is_bf16) {
     if (v) { ELL_MOE_ROWS(__nv_bfloat16, true) } else { ELL_MOE_ROWS(__nv_bfloat16, false) }

@@ -38,7 +38,7 @@ def lib():
             raise KernelError(f"{_LIB_PATH} is missing: run `python -m easyllm_b200.ops.build` "
                               "(or __graft_entry__.build()) before using the CUDA ops")
         _lib = ctypes.CDLL(_LIB_PATH if os.path.exists(_LIB_PATH) else _SERVE_LIB_PATH)
-        for name in ("ell_rmsnorm_bwd_scratch_elems", "ell_attn_rows_scratch"):
+        for name in ("ell_rmsnorm_bwd_scratch_elems", "ell_attn_rows_scratch", "ell_attn_latent_scratch"):
             getattr(_lib, name).restype = c_longlong
     return _lib
 
@@ -503,10 +503,11 @@ def _slopes(alibi_slopes, Hq, device):
     return sl
 
 
-def flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes=None, sink=None):
+def flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes=None, sink=None, window=None):
     """q [T,Hq,D], k [T,Hk,D], v [T,Hk,Dv] (heads packed in a row, any row stride; D and Dv multiples of 8 up to 128)
     → (out [T,Hq,Dv], lse [Hq,T]).  ``alibi_slopes`` fp32 [Hq]: adds ``slope_h · (key − query)`` to the scores;
-    ``sink`` fp32 [Hq]: one more term ``exp(sink_h)`` of the softmax denominator (part of lse)."""
+    ``sink`` fp32 [Hq]: one more term ``exp(sink_h)`` of the softmax denominator (part of lse); ``window``: a row sees its
+    own and the ``window - 1`` keys before it (None: all of its document before it)."""
     T, Hq, D = q.shape
     Hk, Dv = k.shape[1], v.shape[2]
     for t, n in ((q, "q"), (k, "k"), (v, "v")):
@@ -521,7 +522,7 @@ def flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes=None, sink=None):
     sl = _slopes(alibi_slopes, Hq, q.device)
     rc = lib().ell_flash_attn_fwd(_p(q), _p(k), _p(v), _p(out), _p(lse), _p(row_start), c_int(T), c_int(Hq), c_int(Hk),
                                   c_int(D), c_int(Dv), c_int(q.stride(0)), c_int(k.stride(0)), c_int(v.stride(0)),
-                                  c_float(scale), _p(sl), _p(sink), _p(err_flag(q.device)), _stream())
+                                  c_float(scale), _p(sl), _p(sink), c_int(window or 0), _p(err_flag(q.device)), _stream())
     _check(rc, "flash_attn_fwd")
     return out, lse
 

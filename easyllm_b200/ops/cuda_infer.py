@@ -101,6 +101,17 @@ def linear_batch(xs, w):
     return y
 
 
+def head_products(x, w, out):
+    (T, H, K), N = x.shape, w.shape[1]
+    if w.shape != (H, N, K) or not w.is_contiguous() or x.stride(2) != 1 or out.stride(2) != 1 or out.shape != (T, H, N) or \
+            not x.dtype == w.dtype == out.dtype:
+        raise ValueError("head_products: x [T, H, K], a contiguous w [H, N, K] and out [T, H, N] of one dtype")
+    _check(lib().ell_matvec(_p(x), _p(w), _p(None), _p(out), c_longlong(x.stride(1)), c_longlong(N * K),
+                            c_longlong(out.stride(1)), c_int(H), c_int(T), c_int(N), c_int(K), c_int(x.stride(0)),
+                            c_int(out.stride(0)), c_int(0), c_int(0), c_int(0), _bf(x.dtype), _stream()), "head_products")
+    return out
+
+
 def linear_add_(acc, x, w):
     _f32(acc, "acc")
     ldx, M, N = _rows(x, "x"), x.shape[0], w.shape[0]
@@ -122,6 +133,33 @@ def embed_scaled(ids, table, scale):
                                   c_longlong(table.shape[0]), c_float(scale), _bf(table.dtype), _p(err_flag(table.device)),
                                   _stream()), "embed_scaled")
     return out
+
+
+def embed_pairs(ids, table, pairs, scale, mul_prev, mul_cur, row_start, kv_base=None, kv_len=None, hist=None):
+    ids = ids.reshape(-1).to(torch.int64).contiguous()
+    n, W = ids.numel(), table.shape[1]
+    if pairs.shape[1] != W or pairs.dtype != table.dtype or not (table.is_contiguous() and pairs.is_contiguous()):
+        raise ValueError("embed_pairs: two contiguous tables of one width and dtype")
+    if row_start.dtype != torch.int32 or (hist is not None and hist.dtype != torch.int32):
+        raise ValueError("embed_pairs: int32 row_start and token history")
+    out = torch.empty(n, W, dtype=torch.float32, device=table.device)
+    _check(lib().ell_embed_pairs(_p(ids), _p(table), _p(pairs), _p(out), _p(row_start), _p(kv_base), _p(kv_len), _p(hist),
+                                 c_int(n), c_int(W), c_longlong(table.shape[0]), c_longlong(pairs.shape[0] - 1),
+                                 c_longlong(mul_prev), c_longlong(mul_cur), c_float(scale), _bf(table.dtype),
+                                 _p(err_flag(table.device)), _stream()), "embed_pairs")
+    return out
+
+
+def layer_norms(x, weights, eps, out_dtype):
+    _f32(x, "x")
+    n, W = x.shape
+    ys = [torch.empty(n, W, dtype=out_dtype, device=x.device) for _ in weights]
+    if not 1 <= len(weights) <= 2 or any(w.numel() != W for w in weights):
+        raise ValueError("layer_norms: one or two weights of the row's length")
+    w = [_f32(t, "weight") for t in weights] + [None]
+    _check(lib().ell_layer_norms(_p(x), _p(w[0]), _p(w[1]), _p(ys[0]), _p(ys[-1]), c_int(n), c_int(W), c_float(eps),
+                                 _bf(out_dtype), _stream()), "layer_norms")
+    return ys
 
 
 def dynamic_tanh(x, alpha, w, b, out_dtype, add=None):
@@ -170,23 +208,83 @@ def kv_append(kcache, vcache, k, v, base, length):
                                c_int(_heads(v, "v")), _bf(k.dtype), _stream()), "kv_append")
 
 
-def attention_rows(q, k, v, base, length, max_len, scale, sink=None, alibi_slopes=None):
+def _gate(gate, like):
+    """(gate, row stride) as kernel arguments: rows of the activations' dtype."""
+    if gate is None:
+        return _p(None), c_int(0)
+    if gate.dtype != like.dtype:
+        raise ValueError("the output gate must have the activations' dtype")
+    return _p(gate), c_int(_rows(gate, "gate"))
+
+
+def attention_rows(q, k, v, base, length, max_len, scale, sink=None, alibi_slopes=None, window=None, gate=None):
     T, H, d = q.shape
     G, dv = k.shape[1], v.shape[2]
+    max_len = min(max_len, window) if window else max_len
     out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
     need = lib().ell_attn_rows_scratch(c_int(T), c_int(H), c_int(G), c_int(dv), c_int(max_len))
     part = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
     sl = cu._slopes(alibi_slopes, H, q.device)
     _check(lib().ell_attn_rows(_p(q), _p(k), _p(v), _p(out), _p(part), _p(base), _p(length),
-                               _p(None if sink is None else _f32(sink, "sink")), _p(sl), c_int(T), c_int(H), c_int(G),
-                               c_int(d), c_int(dv), c_int(_heads(q, "q")), c_int(_heads(k, "k")), c_int(_heads(v, "v")),
-                               c_int(max_len), c_float(scale), _bf(q.dtype), _stream()), "attn_rows", 2 if need else 1)
+                               _p(None if sink is None else _f32(sink, "sink")), _p(sl), _gate(gate, q)[0], c_int(T),
+                               c_int(H), c_int(G), c_int(d), c_int(dv), c_int(_heads(q, "q")), c_int(_heads(k, "k")),
+                               c_int(_heads(v, "v")), _gate(gate, q)[1], c_int(max_len), c_int(window or 0), c_float(scale),
+                               _bf(q.dtype), _stream()), "attn_rows", 2 if need else 1)
     return out
 
 
-def attention_prefill(q, k, v, row_start, scale, sink=None, alibi_slopes=None):
+def attention_prefill(q, k, v, row_start, scale, sink=None, alibi_slopes=None, window=None):
     """Packed prompts on the tcgen05 kernel (bf16, heads of up to 128)."""
-    return cu.flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes, sink)[0]
+    return cu.flash_attn_fwd(q, k, v, row_start, scale, alibi_slopes, sink, window)[0]
+
+
+# ---- latent attention ------------------------------------------------------------------------------
+def latent_inputs(z, H, dim, rot, rank, norm_w, eps, cos, sin, meta, cache=None, q_dst=None):
+    n, ldz = z.shape[0], _rows(z, "z") and z.stride(0)
+    pos = meta["position_ids"]
+    if pos.dtype != torch.int32 or cos.shape != sin.shape or not (_f32(cos, "cos") is cos and _f32(sin, "sin") is sin):
+        raise ValueError("latent_inputs: int32 positions, fp32 angle tables")
+    if z.shape[1] < H * (dim + rot) + rank + rot or norm_w.numel() != rank:
+        raise ValueError("latent_inputs: the rows hold H (dim + rot) + rank + rot columns")
+    if cache is not None and (cache.dtype != z.dtype or not cache.is_contiguous() or cache.shape[-1] < rank + rot):
+        raise ValueError("latent_inputs: a contiguous cache of the activations' dtype")
+    if q_dst is not None and (q_dst.dtype != z.dtype or q_dst.stride(2) != 1 or
+                              (n > 1 and q_dst.stride(0) != H * q_dst.stride(1))):
+        raise ValueError("latent_inputs: q_dst must be a slice of packed heads")
+    _check(lib().ell_latent_inputs(_p(z), _p(q_dst), _p(cache), _p(_f32(norm_w, "norm")), _p(cos), _p(sin), _p(pos),
+                                   _p(None if cache is None else meta["kv_base"]),
+                                   _p(None if cache is None else meta["kv_len"]), c_int(n), c_int(H), c_int(dim), c_int(rot),
+                                   c_int(rank), c_int(cos.shape[1]), c_int(ldz), c_int(0 if q_dst is None else q_dst.stride(1)),
+                                   c_int(0 if cache is None else cache.shape[-1]), c_float(eps), _bf(z.dtype), _stream()),
+           "latent_inputs")
+
+
+def attention_latent(q, rows, dv, base, length, max_len, scale, window=None, gate=None):
+    T, H, d = q.shape
+    ldk = _rows(rows, "rows")
+    if rows.dtype != q.dtype or rows.shape[1] < d or dv > d:
+        raise ValueError("attention_latent: key rows of the queries' dtype and size")
+    out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
+    shape = (c_int(T), c_int(H), c_int(d), c_int(dv), c_int(_heads(q, "q")), c_int(ldk))
+    need = lib().ell_attn_latent_scratch(*shape, c_int(max_len), c_int(window or 0), _bf(q.dtype))
+    part = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
+    g, ldg = _gate(gate, q)
+    _check(lib().ell_attn_latent(_p(q), _p(rows), _p(out), _p(part), _p(base), _p(length), g, *shape, ldg, c_int(max_len),
+                                 c_int(window or 0), c_float(scale), _bf(q.dtype), _stream()), "attn_latent", 2 if need else 1)
+    return out
+
+
+def attention_latent_prefill(z, kv, H, dim, rot, rank, vdim, row_start, scale, window=None, gate=None):
+    T, at = z.shape[0], H * (dim + rot)
+    out = torch.empty(T, H, vdim, dtype=z.dtype, device=z.device)
+    k2, v = z[:, at + rank:], kv[:, H * dim:]
+    g, ldg = _gate(gate, z)
+    ldz, ldkv = _rows(z, "z") and z.stride(0), _rows(kv, "kv")
+    _check(lib().ell_flash_attn_latent(_p(z), _p(kv), _p(k2), _p(v), _p(out), _p(row_start), g, c_int(T), c_int(H), c_int(dim),
+                                       c_int(rot), c_int(vdim), c_int(ldz), c_int(ldkv), c_int(ldz), c_int(ldkv), ldg,
+                                       c_int(window or 0), c_float(scale), _p(err_flag(z.device)), _stream()),
+           "flash_attn_latent")
+    return out
 
 
 # ---- recurrences -----------------------------------------------------------------------------------
@@ -271,40 +369,49 @@ def head_norm_gate(o, w, gate, gate_act, eps, out_dtype):
 
 
 # ---- mixture of experts ------------------------------------------------------------------------------
-def moe_route(z, top):
-    """fp32 router logits ``[T, E]`` → (expert int32 ``[T, top]``, sigmoid score fp32 ``[T, top]``)."""
+def moe_route(z, top, bias=None, softmax=False):
+    """fp32 router logits ``[T, E]`` (plus ``bias [E]``) → (expert int32 ``[T, top]``, fp32 ``[T, top]``: sigmoid scores, or
+    the softmax over the chosen logits)."""
     T, E = z.shape
     idx = torch.empty(T, top, dtype=torch.int32, device=z.device)
     w = torch.empty(T, top, dtype=torch.float32, device=z.device)
     if z.dtype != torch.float32:
         raise ValueError("moe_route: fp32 logits")
-    _check(lib().ell_moe_route(_p(z), _p(idx), _p(w), c_int(T), c_int(E), c_int(top), c_int(_rows(z, "z")), _stream()),
-           "moe_route")
+    _check(lib().ell_moe_route(_p(z), _p(None if bias is None else _f32(bias, "bias")), _p(idx), _p(w), c_int(T), c_int(E),
+                               c_int(top), c_int(_rows(z, "z")), c_int(softmax), _stream()), "moe_route")
     return idx, w
 
 
 def moe_relu2_add_(acc, h, z, top, up, down):
+    return _moe_add_(acc, h, *moe_route(z, top), up, down)
+
+
+def moe_glu_add_(acc, h, z, bias, top, gate_up, block, down):
+    return _moe_add_(acc, h, *moe_route(z, top, bias, softmax=True), gate_up, down, block)
+
+
+def _moe_add_(acc, h, idx, w, up, down, block=0):
+    """``block`` 0: two-matrix experts; otherwise ``up`` holds gate and up rows in alternating blocks of that many."""
     _f32(acc, "acc")
     h = h.contiguous()
     T, W = h.shape
-    E, F = up.shape[:2]
-    idx, w = moe_route(z, top)
-    if h.dtype == torch.bfloat16 and T * top > max(MATVEC_ROWS, 2 * E) and W % 8 == 0 and F % 8 == 0:
-        return _moe_grouped(acc, h, idx, w, up, down)
+    E, F, top = up.shape[0], down.shape[2], idx.shape[1]
+    if h.dtype == torch.bfloat16 and T * top > max(MATVEC_ROWS, 2 * E) and W % 8 == 0 and F % 8 == 0 and block in (0, 32):
+        return _moe_grouped(acc, h, idx, w, up, down, block)
     step = max(1, 65535 // top)
     for t in range(0, T, step):                         # the slots are a grid dimension
         n = min(step, T - t)
         hid = torch.empty(n * top, F, dtype=h.dtype, device=h.device)
         _check(lib().ell_moe_rows(_p(h[t:]), _p(up), _p(down), _p(idx[t:]), _p(w[t:]), _p(hid), _p(acc[t:]), c_int(n),
-                                  c_int(top), c_int(F), c_int(W), _bf(h.dtype), _stream()), "moe_rows", 2)
+                                  c_int(top), c_int(F), c_int(W), c_int(block), _bf(h.dtype), _stream()), "moe_rows", 2)
     return acc
 
 
-def _moe_grouped(acc, h, idx, w, up, down):
-    """Rows sorted by expert, two grouped tcgen05 GEMMs (the squared relu with the routing weight in the first one's
+def _moe_grouped(acc, h, idx, w, up, down, block=0):
+    """Rows sorted by expert, two grouped tcgen05 GEMMs (the activation with the routing weight in the first one's
     epilogue), and the sum back into ``acc``.  The row plan stays on the device."""
     T, W = h.shape
-    E, F = up.shape[:2]
+    E, F = up.shape[0], down.shape[2]
     top, dev = idx.shape[1], h.device
     used = min(E, T * top)                              # experts that can have rows
     tiles = (T * top - used) // 128 + used              # most 128-row tiles any routing can need
@@ -317,8 +424,9 @@ def _moe_grouped(acc, h, idx, w, up, down):
                                 c_int(top), c_int(E), c_int(W), _stream()), "moe_gather", 2)
     hid = torch.empty(rows, F, dtype=h.dtype, device=dev)
     ys = torch.empty(rows, W, dtype=h.dtype, device=dev)
-    for x, wt, out, n, k, sc in ((xs, up, hid, F, W, scale), (hid, down, ys, W, F, None)):
+    for x, wt, out, n, k, sc in ((xs, up, hid, up.shape[1], W, scale), (hid, down, ys, W, F, None)):
         _check(lib().ell_gemm_grouped(_p(x), _p(wt), _p(out), _p(tile_expert), _p(n_tiles), _p(sc), c_int(rows), c_int(n),
-                                      c_int(k), c_int(E), _p(err_flag(dev)), _stream()), "gemm_grouped")
+                                      c_int(k), c_int(E), c_int(bool(block) and sc is not None), _p(err_flag(dev)), _stream()),
+               "gemm_grouped")
     _check(lib().ell_moe_combine(_p(ys), _p(pos), _p(acc), c_int(T), c_int(top), c_int(W), _stream()), "moe_combine")
     return acc

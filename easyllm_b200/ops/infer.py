@@ -112,12 +112,46 @@ def linear_add_(acc, x, w):
     return acc.add_(F.linear(x, w).float())
 
 
+def head_products(x, w, out=None):
+    """Per head ``x[:, h] W_hᵀ``: x ``[T, H, K]``, w ``[H, N, K]`` → ``[T, H, N]`` (``out``: may be a slice of wider rows)."""
+    if out is None:
+        out = torch.empty(x.shape[0], w.shape[0], w.shape[1], dtype=x.dtype, device=x.device)
+    if _kern(x):
+        return _cu().head_products(x, w, out)
+    out.copy_(torch.einsum("thk,hnk->thn", x, w))
+    return out
+
+
 # ---- elementwise -------------------------------------------------------------------------------
 def embed_scaled(ids, table, scale):
     """fp32 ``table[ids] * scale``."""
     if _kern(table):
         return _cu().embed_scaled(ids, table.detach(), scale)
     return F.embedding(ids, table).float() * scale
+
+
+def row_start(meta, n, device):
+    """Row of the first token of each token's sequence in this batch."""
+    if meta.get("row_start") is not None:
+        return meta["row_start"]
+    cu = meta["cu_seqlens"].long()
+    return torch.repeat_interleave(cu[:-1], cu[1:] - cu[:-1], output_size=n).to(device=device, dtype=torch.int32)
+
+
+def embed_pairs(ids, table, pairs, scale, mul_prev, mul_cur, meta, hist=None):
+    """Embedding plus a table of (previous token, token) pairs, see ``reference_infer.embed_pairs``.  ``hist``: the state's
+    token ids ``[slots, capacity]``, or None."""
+    no_grad_check(table, pairs)
+    start = row_start(meta, ids.numel(), ids.device)
+    place = (meta["kv_base"], meta["kv_len"], hist.view(-1)) if hist is not None else (None, None, None)
+    f = _cu().embed_pairs if _kern(table) else ref.embed_pairs
+    return f(ids, table.detach(), pairs.detach(), scale, mul_prev, mul_cur, start, *place)
+
+
+def layer_norms(x, weights, eps, out_dtype):
+    """Layer norms of one fp32 ``x`` with one or two weights and no bias; the statistics are taken once."""
+    ws = [w.detach() for w in weights]
+    return _cu().layer_norms(x, ws, eps, out_dtype) if x.is_cuda else ref.layer_norms(x, ws, eps, out_dtype)
 
 
 def dynamic_tanh(x, alpha, w, b, out_dtype, add=None):
@@ -154,12 +188,12 @@ def kv_append(kcache, vcache, k, v, meta):
     vcache.view(-1, *vcache.shape[2:])[rows] = v
 
 
-def attention_rows(q, k, v, kv_base, kv_len, max_len, scale, sink=None, alibi_slopes=None):
+def attention_rows(q, k, v, kv_base, kv_len, max_len, scale, sink=None, alibi_slopes=None, window=None, gate=None):
     """Causal attention of query rows over key/value rows (a cache, or the packed batch itself), see
     ``reference_infer.attention_rows``.  ``max_len`` bounds ``kv_len``."""
     if _kern(q):
-        return _cu().attention_rows(q, k, v, kv_base, kv_len, max_len, scale, sink, alibi_slopes)
-    return ref.attention_rows(q, k, v, kv_base, kv_len, scale, sink, alibi_slopes)
+        return _cu().attention_rows(q, k, v, kv_base, kv_len, max_len, scale, sink, alibi_slopes, window, gate)
+    return ref.attention_rows(q, k, v, kv_base, kv_len, scale, sink, alibi_slopes, window, gate)
 
 
 def prefill_kernel_ok(q, v):
@@ -168,8 +202,43 @@ def prefill_kernel_ok(q, v):
         q.shape[-1] % 8 == 0 and v.shape[-1] % 8 == 0
 
 
-def attention_prefill(q, k, v, row_start, scale, sink=None, alibi_slopes=None):
-    return _cu().attention_prefill(q, k, v, row_start, scale, sink, alibi_slopes)
+def attention_prefill(q, k, v, row_start, scale, sink=None, alibi_slopes=None, window=None):
+    return _cu().attention_prefill(q, k, v, row_start, scale, sink, alibi_slopes, window)
+
+
+# ---- latent attention ------------------------------------------------------------------------------
+def latent_inputs(z, H, dim, rot, rank, norm_w, eps, cos, sin, meta, cache=None, q_dst=None):
+    """Rotations and latent norm on the projection rows, in place, see ``reference_infer.latent_inputs``.  ``cache
+    [slots, capacity, ld]`` receives latent and rotated key part of the step's tokens."""
+    if _kern(z):
+        return _cu().latent_inputs(z, H, dim, rot, rank, norm_w.detach(), eps, cos, sin, meta, cache, q_dst)
+    pos = meta["position_ids"].long()
+    ref.latent_inputs(z, H, dim, rot, rank, norm_w, eps, cos[pos], sin[pos], q_dst)
+    if cache is not None:
+        rows = (meta["kv_base"] + meta["kv_len"] - 1).long()
+        at = H * (dim + rot)
+        cache.view(-1, cache.shape[-1])[rows, :rank + rot] = z[:, at:at + rank + rot]
+
+
+def attention_latent(q, rows, dv, kv_base, kv_len, max_len, scale, window=None, gate=None):
+    """Attention in the latent space: q ``[T, H, d]`` over one key row ``rows[:, :d]`` per position, shared by all heads,
+    whose first ``dv`` columns are the value → ``[T, H, dv]``.  Places as in ``attention_rows``."""
+    if _kern(q):
+        return _cu().attention_latent(q, rows, dv, kv_base, kv_len, max_len, scale, window, gate)
+    k = rows[:, :q.shape[-1]].unsqueeze(1)
+    return ref.attention_rows(q, k, k[..., :dv], kv_base, kv_len, scale, window=window, gate=gate)
+
+
+def latent_prefill_ok(z, dim, rot, rank, vdim):
+    """Whether the tcgen05 attention kernel takes packed prompts with keys of these two parts."""
+    return z.is_cuda and z.dtype == torch.bfloat16 and not (dim % 8 or rot % 8 or vdim % 8 or rank % 8) and min(dim, rot) > 0 \
+        and -(-dim // 64) + -(-rot // 64) <= 3 and vdim <= 128 and z.stride(0) % 8 == 0
+
+
+def attention_latent_prefill(z, kv, H, dim, rot, rank, vdim, row_start, scale, window=None, gate=None):
+    """Packed prompts: queries and the shared key part from the projection rows ``z``, the heads' own key parts and values
+    from ``kv [T, H dim + H vdim]`` → ``[T, H, vdim]``."""
+    return _cu().attention_latent_prefill(z, kv, H, dim, rot, rank, vdim, row_start, scale, window, gate)
 
 
 # ---- recurrences -----------------------------------------------------------------------------------
@@ -223,3 +292,14 @@ def moe_relu2_add_(acc, h, z, top, up, down):
         return _cu().moe_relu2_add_(acc, h, z, top, up.detach(), down.detach())
     idx, w = ref.route(z, top)
     return acc.add_(ref.moe_relu2(h, idx, w, up, down))
+
+
+def moe_glu_add_(acc, h, z, bias, top, gate_up, block, down):
+    """``acc += sum over the top experts of w_e down_e (silu(gate_e h) * up_e h)``, ``w`` the softmax over the chosen logits
+    of ``z + bias``; gate_up ``[E, 2 F, W]`` holds gate and up rows in alternating blocks of ``block``."""
+    no_grad_check(h, gate_up)
+    bias = None if bias is None else bias.detach()
+    if _kern(h):
+        return _cu().moe_glu_add_(acc, h, z, bias, top, gate_up.detach(), block, down.detach())
+    idx, w = ref.route_softmax(z, bias, top)
+    return acc.add_(ref.moe_glu(h, idx, w, gate_up, block, down))

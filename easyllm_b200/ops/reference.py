@@ -46,6 +46,33 @@ def rope_tables(head_dim, max_pos, base=10000.0, scale_factor=1.0, device=None, 
     return fr.cos(), fr.sin()
 
 
+def yarn_frequencies(dims, base, scaling=None):
+    """Angular frequency of every rotated pair and the factor of cos and sin, in double precision.
+
+    ``scaling`` (None: the plain ``base ** (-2 i / dims)``): a dict with ``factor`` and ``original`` (the context length the
+    frequencies were made for).  Pairs that turn more than ``fast`` times over that length keep their frequency, those that
+    turn less than ``slow`` times are slowed down by ``factor``, with a linear ramp between; cos and sin grow by
+    ``0.1 ln(factor) + 1``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = base ** (-2 * i / dims)
+    if not scaling:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def at(turns):
+        return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(at(scaling["fast"])), 0), min(math.ceil(at(scaling["slow"])), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f / factor * ramp + f * (1 - ramp), 0.1 * math.log(factor) + 1
+
+
+def yarn_tables(dims, max_pos, base, scaling=None, device=None):
+    """fp32 cos/sin tables ``[max_pos, dims/2]`` of ``yarn_frequencies``; the angles are formed in double precision."""
+    f, m = yarn_frequencies(dims, base, scaling)
+    a = torch.outer(torch.arange(max_pos, dtype=torch.float64), f)
+    return (a.cos() * m).float().to(device), (a.sin() * m).float().to(device)
+
+
 def rope(q, k, cos, sin, position_ids):
     """Apply rotary embedding to ``q [T,Hq,D]`` and ``k [T,Hk,D]``; ``position_ids [T]`` int."""
     c = cos[position_ids].unsqueeze(1)

@@ -28,9 +28,56 @@ def _segments(cu, slots, pos0):
             yield cu[s], cu[s + 1], slot, fresh
 
 
-def attention_rows(q, k, v, kv_base, kv_len, scale, sink=None, alibi_slopes=None):
+def embed_pairs(ids, table, pairs, scale, mul_prev, mul_cur, row_start, kv_base=None, kv_len=None, hist=None):
+    """fp32 ``table[id] * scale + pairs[(previous id * mul_prev + id * mul_cur) mod buckets]``, ``buckets`` one less than the
+    rows of ``pairs``; a sequence's first token takes the last row.  ``hist``: token ids by position (flat), the previous
+    token of a sequence's first row in this step; this step's ids are written to it."""
+    t = torch.arange(ids.numel())
+    first = row_start.cpu() == t
+    prev = ids.roll(1).clone()
+    buckets = pairs.shape[0] - 1
+    if hist is not None:
+        at = (kv_base + kv_len - 1).long()
+        going_on = first & (kv_len.cpu() > 1)
+        prev[going_on] = hist[at[going_on] - 1].to(prev.dtype)
+        first = first & ~going_on
+        hist[at] = ids.to(hist.dtype)
+    row = torch.where(first.to(ids.device), buckets, (prev * mul_prev + ids * mul_cur) % buckets)
+    return table[ids].float() * scale + pairs[row].float()
+
+
+def layer_norms(x, weights, eps, out_dtype):
+    """``(x - mean) / sqrt(variance + eps) * w`` for every ``w``."""
+    d = x.float() - x.float().mean(-1, keepdim=True)
+    y = d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps)
+    return [(y * w.float()).to(out_dtype) for w in weights]
+
+
+def rotate_pairs(x, cos, sin):
+    """x ``[T, n, r]`` with neighbouring dimensions as pairs, cos / sin ``[T, pairs]``; dimensions past them stay."""
+    n = 2 * cos.shape[-1]
+    u, v = x[..., :n:2].float(), x[..., 1:n:2].float()
+    c, s = cos.unsqueeze(1), sin.unsqueeze(1)
+    y = torch.stack((u * c - v * s, v * c + u * s), -1).flatten(-2).to(x.dtype)
+    return torch.cat((y, x[..., n:]), -1)
+
+
+def latent_inputs(z, H, dim, rot, rank, norm_w, eps, cos, sin, q_dst=None):
+    """In place on ``z [T, H (dim + rot) + rank + rot + ...]``: the rotated query parts (into ``q_dst [T, H, rot]`` if
+    given), the latent over its root mean square times ``norm_w``, the rotated key part."""
+    T, at = z.shape[0], H * (dim + rot)
+    q = z[:, :at].view(T, H, dim + rot)
+    (q[..., dim:] if q_dst is None else q_dst).copy_(rotate_pairs(q[..., dim:], cos, sin))
+    c = z[:, at:at + rank].float()
+    z[:, at:at + rank] = (c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()).to(z.dtype)
+    kr = z[:, at + rank:at + rank + rot]
+    kr.copy_(rotate_pairs(kr.unsqueeze(1), cos, sin).squeeze(1))
+
+
+def attention_rows(q, k, v, kv_base, kv_len, scale, sink=None, alibi_slopes=None, window=None, gate=None):
     """Query row t attends to the rows ``kv_base[t] .. kv_base[t] + kv_len[t]`` of k ``[R, G, d]``, v ``[R, G, dv]``;
-    it sits at the last of them.  ``sink [H]`` adds ``exp(sink)`` to the softmax denominator."""
+    it sits at the last of them.  ``sink [H]`` adds ``exp(sink)`` to the softmax denominator; ``window`` keeps the last so
+    many rows; ``gate [T, H]`` multiplies the heads' outputs by its sigmoid."""
     T, H, _ = q.shape
     G, dv = k.shape[1], v.shape[2]
     out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
@@ -49,11 +96,12 @@ def attention_rows(q, k, v, kv_base, kv_len, scale, sink=None, alibi_slopes=None
         kj = torch.arange(n, device=q.device).view(1, -1)
         if alibi_slopes is not None:
             s = s + alibi_slopes.float().view(-1, 1, 1) * (kj - qi)
-        s = s.masked_fill(kj > qi, float("-inf"))
+        s = s.masked_fill((kj > qi) | (kj <= qi - window) if window else kj > qi, float("-inf"))
         if sink is not None:
             s = torch.cat((s, sink.float().view(H, 1, 1).expand(H, e - t, 1)), -1)
         p = torch.softmax(s, -1)[..., :n]
-        out[t:e] = torch.einsum("hqk,khd->qhd", p, vs).to(q.dtype)
+        o = torch.einsum("hqk,khd->qhd", p, vs)
+        out[t:e] = (o if gate is None else o * torch.sigmoid(gate[t:e].float()).unsqueeze(-1)).to(q.dtype)
         t = e
     return out
 
@@ -148,6 +196,30 @@ def route(z, top):
     s = torch.sigmoid(z.float())
     w, idx = torch.topk(s, top, dim=-1)
     return idx, w
+
+
+def route_softmax(z, bias, top):
+    """Router logits plus ``bias`` → (the ``top`` largest per token, the softmax over them)."""
+    w, idx = torch.topk(z.float() if bias is None else z.float() + bias.float(), top, dim=-1)
+    return idx, torch.softmax(w, -1)
+
+
+def unblock(gate_up, block):
+    """``[..., 2 F, W]`` with gate and up rows in alternating blocks → gate, up ``[..., F, W]``."""
+    F_, W = gate_up.shape[-2] // 2, gate_up.shape[-1]
+    v = gate_up.view(*gate_up.shape[:-2], F_ // block, 2, block, W)
+    return v[..., 0, :, :].reshape(*gate_up.shape[:-2], F_, W), v[..., 1, :, :].reshape(*gate_up.shape[:-2], F_, W)
+
+
+def moe_glu(h, idx, weight, gate_up, block, down):
+    """sum over the chosen experts of ``w down_e (silu(gate_e h) * up_e h)`` → fp32; the weight joins the hidden units."""
+    gate, up = unblock(gate_up, block)
+    out = torch.zeros(h.shape[0], down.shape[1], dtype=torch.float32, device=h.device)
+    for e in idx.unique().tolist():
+        t, s = torch.nonzero(idx == e, as_tuple=True)
+        a = F.silu(F.linear(h[t], gate[e]).float()) * F.linear(h[t], up[e]).float() * weight[t, s].unsqueeze(-1)
+        out.index_add_(0, t, F.linear(a.to(h.dtype), down[e]).float())
+    return out
 
 
 def moe_relu2(h, idx, weight, up, down):
