@@ -128,14 +128,16 @@ def main():
                     help="packed variable-length documents (lengths uniform in [256, seq]) with cu_seqlens")
     ap.add_argument("--no-fused-tp", action="store_true", help="use the NCCL + GEMM composition for TP linears")
     ap.add_argument("--serving", action="store_true", help="instead of the training step: prompt and decode throughput of "
-                    "the hybrid decoder beside a Llama of equal size (easyllm_b200/infer/bench_serving.py)")
+                    "a hybrid decoder beside the closest model of equal size (easyllm_b200/infer/bench_serving.py)")
+    ap.add_argument("--serving-model", default="pafodra", choices=["pafodra", "megozen"])
     ap.add_argument("--serving-sizes", default="2k,4k")
     ap.add_argument("--serving-kernels", action="store_true", help="with --serving: also every kernel against its roofline")
     args = ap.parse_args()
 
     if args.serving:
         from easyllm_b200.infer import bench_serving
-        return bench_serving.main(args.serving_sizes.split(","), args.serving_kernels, clocks=lambda: ClockSampler(0))
+        return bench_serving.main(args.serving_sizes.split(","), args.serving_kernels, clocks=lambda: ClockSampler(0),
+                                  model=args.serving_model)
 
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":

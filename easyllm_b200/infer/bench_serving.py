@@ -1,7 +1,9 @@
-"""Serving throughput: prompts and decoding of a hybrid decoder (Pafodra) beside a Llama of equal size, and the kernels
-of both one by one against their rooflines.
+"""Serving throughput: prompts and decoding of a hybrid decoder beside the closest other model at equal size, and the
+kernels of both one by one against their rooflines.
 
-    python bench.py --serving [--serving-sizes 2k,4k] [--serving-kernels]
+    python bench.py --serving [--serving-model pafodra|megozen] [--serving-sizes 2k,4k] [--serving-kernels]
+
+Pafodra is measured beside a Llama, Megozen beside a Pafodra of attention layers with experts only.
 
 Random weights; synthetic token ids.  Times are CUDA events on the launching stream, 3 warm-ups, medians.  The models
 (gigabytes of weights) are far larger than L2; single kernels are timed with an L2 flush between iterations.  Prompts go
@@ -36,9 +38,36 @@ def pafodra_config(s):
             "embedding": {"scale": 4.0}, "layers": [period[i % 5] for i in range(s["layers"])]}
 
 
+def pafodra_attention_config(s):
+    """Attention layers with experts only: the closest relative of the Megozen below."""
+    d = 128
+    layer = {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv"], "dim": d, "vdim": d, "scale": d ** -0.5},
+             "mlp": {"kind": "moe", "router": {"experts": s["experts"], "top": 2}, "expert": {"ff": s["eff"]},
+                     "shared": {"ff": s["eff"]}}}
+    return dict(pafodra_config(s), layers=[layer] * s["layers"])
+
+
+# latent attention: heads of 128 unrotated + 64 rotated dimensions over a latent of 512, a window of 1024 tokens
+LATENT = dict(dim=128, rot=64, vdim=128, rank=512, window=1024)
+
+
+def megozen_config(s):
+    m = LATENT
+    rot = {"dims": m["rot"], "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    layer = {"type": "latent_attention",
+             "mixer": {"heads": s["heads"], "dim": m["dim"], "rot_dim": m["rot"], "vdim": m["vdim"], "kv_rank": m["rank"],
+                       "scale": (m["dim"] + m["rot"]) ** -0.5, "rot": rot, "mask": {"size": m["window"]}},
+             "mlp": {"kind": "moe", "router": {"experts": s["experts"], "top": 2}, "expert": {"ff": s["eff"]},
+                     "shared": {"ff": s["eff"]}}}
+    return {"architecture": "Megozen", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": s["vocab"] - 1, "mul_prev": 7919, "mul_cur": 104729}},
+            "layers": [layer] * s["layers"]}
+
+
 def build(which, s):
     from ..models.hf_models import CausalLM, HFArch, arch_from_hf_config
-    arch = arch_from_hf_config(pafodra_config(s)) if which == "pafodra" else HFArch(
+    configs = {"pafodra": pafodra_config, "pafodra attention": pafodra_attention_config, "megozen": megozen_config}
+    arch = arch_from_hf_config(configs[which](s)) if which in configs else HFArch(
         family="llama", vocab_size=s["vocab"], hidden_size=s["width"], intermediate_size=s["ff"],
         num_hidden_layers=s["layers"], num_attention_heads=s["heads"], num_key_value_heads=s["kv"])
     torch.manual_seed(0)
@@ -185,14 +214,105 @@ def kernel_cases(s, T, B, context):
     del ops
 
 
+def megozen_cases(s, T, B, context):
+    """As ``kernel_cases``: Megozen's kernels, each followed by the like one of the other decoders."""
+    from ..models.hf_models.feedforward import SparseGLU
+    from ..models.layers import YarnRotaryTables
+    from ..ops import cuda as cu
+    from ..ops import cuda_infer as ci
+    W, H, G, E, EF, V = s["width"], s["heads"], s["kv"], s["experts"], s["eff"], s["vocab"]
+    d, r, dv, R, win = (LATENT[k] for k in ("dim", "rot", "vdim", "rank", "window"))
+    bf, f32, dev = torch.bfloat16, torch.float32, "cuda"
+    at, D = H * (d + r), 128
+
+    def rnd(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(*shape, device=dev) * scale).to(dtype)
+    cos, sin = YarnRotaryTables(r, 1e4).get(context, torch.device(dev))
+    for phase, n in (("prefill", T), ("decode", B)):
+        x32, h = rnd(n, W, dtype=f32), rnd(n, W)
+        w1, w2, al = rnd(W, dtype=f32), rnd(W, dtype=f32), torch.tensor(0.5, device=dev)
+        pos = torch.arange(n, device=dev, dtype=torch.int32) % context
+        m = {"position_ids": pos, "kv_base": torch.zeros(n, dtype=torch.int32, device=dev) if phase == "prefill" else
+             torch.arange(0, n * context, context, dtype=torch.int32, device=dev), "kv_len": pos + 1}
+        start = torch.zeros(n, dtype=torch.int32, device=dev)
+        ids, table, pairs = torch.randint(0, V, (n,), device=dev), rnd(V, W), rnd(V, W)
+        yield "layer_norms (two)", phase, lambda: ci.layer_norms(x32, [w1, w2], 1e-6, bf), 8 * n * W, 0, 0
+        yield "like: dynamic_tanh", phase, lambda: ci.dynamic_tanh(x32, al, w1, w2, bf), 6 * n * W, 0, 0
+        yield "embed_pairs", phase, lambda: ci.embed_pairs(ids, table, pairs, 1.0, 7919, 104729, start), 8 * n * W, 0, 0
+        yield "like: embed_scaled", phase, lambda: ci.embed_scaled(ids, table, 2.0), 6 * n * W, 0, 0
+        N = at + R + r + H
+        win_, wq = rnd(N, W, scale=0.02), rnd((H + 2 * G) * D, W, scale=0.02)
+        yield "linear q|latent|gate", phase, lambda: ci.linear(h, win_), 2 * (n * W + N * W + n * N), 2 * n * N * W, 0
+        yield ("like: linear qkv", phase, lambda: ci.linear(h, wq), 2 * (n * W + wq.numel() + n * (H + 2 * G) * D),
+               2 * n * wq.numel(), 0)
+        z = ci.linear(h, win_)
+        cache, nw = rnd(max(n if phase == "decode" else 1, 1), context, R + r), rnd(R, dtype=f32)
+        q = rnd(n, H, R + r)
+        moved = n * (4 * H * r + 6 * (R + r))
+        yield ("latent_inputs", phase, lambda: ci.latent_inputs(z, H, d, r, R, nw, 1e-6, cos, sin, m, cache,
+                                                                q[..., R:] if phase == "decode" else None), moved, 0, 0)
+        qkv = rnd(n, 3 * H * D)
+        c2, s2 = YarnRotaryTables(D, 1e4).get(context, torch.device(dev))
+        yield ("like: rope of q and k", phase, lambda: cu.rope_(qkv, c2, s2, pos, 2 * H, D), n * 2 * H * D * 4, 0, 0)
+        gu = torch.stack([SparseGLU.blocked(rnd(EF, W, scale=0.02), rnd(EF, W, scale=0.02)) for _ in range(E)])
+        down, up = rnd(E, W, EF, scale=0.02), rnd(E, EF, W, scale=0.02)
+        zr, hit = rnd(n, E, dtype=f32), min(E, 2 * n)
+        yield ("gated experts (all launches)", phase, lambda: ci.moe_glu_add_(x32, h, zr, None, 2, gu, 32, down),
+               2 * 3 * hit * EF * W + 2 * n * W + 8 * n * W, 2 * 2 * n * 3 * EF * W, 0)
+        yield ("like: experts (all launches)", phase, lambda: ci.moe_relu2_add_(x32, h, zr, 2, up, down),
+               2 * 2 * hit * EF * W + 2 * n * W + 8 * n * W, 2 * 2 * n * 2 * EF * W, 0)
+        sg, wo, o = rnd(n, 2 * EF), rnd(W, H * dv, scale=0.02), rnd(n, H * dv)
+        yield "glu silu (shared expert)", phase, lambda: ci.glu(sg, "silu"), 6 * n * EF, 0, 0
+        yield "like: glu gelu", phase, lambda: ci.glu(sg, "gelu_tanh"), 6 * n * EF, 0, 0
+        yield ("linear o += fp32", phase, lambda: ci.linear_add_(x32, o, wo), 2 * (n * H * dv + wo.numel()) + 8 * n * W,
+               2 * n * wo.numel(), 0)
+        gate = z[:, at + R + r:]
+        if phase == "prefill":
+            wkv = rnd(H * (d + dv), R, scale=0.04)
+            yield ("linear latent -> k|v", phase, lambda: ci.linear(z[:, at:at + R], wkv),
+                   2 * (n * R + wkv.numel() + n * H * (d + dv)), 2 * n * wkv.numel(), 0)
+            kv = ci.linear(z[:, at:at + R], wkv)
+            for w, seen in ((win, n * win - win * (win - 1) / 2), (None, n * (n + 1) / 2)):
+                yield (f"latent attention, {'window %d' % w if w else 'all keys'}", phase,
+                       lambda: ci.attention_latent_prefill(z, kv, H, d, r, R, dv, start, 0.07, w, gate),
+                       2 * n * (at + R + r + 2 * H * (d + dv)), 2 * seen * H * (d + r + dv), 0)
+            q3, k3, v3, sink = rnd(n, H, D), rnd(n, G, D), rnd(n, G, D), rnd(H, dtype=f32)
+            yield ("like: attention + sink", phase, lambda: ci.attention_prefill(q3, k3, v3, start, 0.09, sink),
+                   2 * n * D * (2 * H + 2 * G), 2 * n * n * D * H, 0)
+        else:
+            ukt, uv = rnd(H, R, d, scale=0.1), rnd(H, dv, R, scale=0.04)
+            qn = z[:, :at].unflatten(1, (H, -1))[..., :d]
+            yield ("query into the latent (per head)", phase, lambda: ci.head_products(qn, ukt, q[..., :R]),
+                   2 * (ukt.numel() + n * H * (d + R)), 2 * n * ukt.numel(), 0)
+            out, lat = torch.empty(n, H, dv, dtype=bf, device=dev), rnd(n, H, R)
+            yield ("latent -> value (per head)", phase, lambda: ci.head_products(lat, uv, out),
+                   2 * (uv.numel() + n * H * (dv + R)), 2 * n * uv.numel(), 0)
+            for b in (1, B, 64):
+                rows = rnd(b * context, R + r)
+                qb, gb = rnd(b, H, R + r), rnd(b, H)
+                base = torch.arange(0, b * context, context, dtype=torch.int32, device=dev)
+                ln = torch.full((b,), context, dtype=torch.int32, device=dev)
+                for w in (None, win):
+                    keys = min(context, w or context)
+                    yield (f"latent attention, batch {b}, {keys} keys", phase,
+                           lambda: ci.attention_latent(qb, rows, R, base, ln, context, 0.07, w, gb),
+                           2 * b * keys * (R + r), 2 * b * H * keys * (2 * R + r), 0)
+                kc, vc, q3 = rnd(b * context, G, D), rnd(b * context, G, D), rnd(b, H, D)
+                yield (f"like: attention rows, batch {b}, {context} keys", phase,
+                       lambda: ci.attention_rows(q3, kc, vc, base, ln, context, 0.09), 4 * b * context * G * D, 0, 0)
+                short = torch.full((b,), win, dtype=torch.int32, device=dev)
+                yield (f"like: attention rows, batch {b}, {win} keys", phase,
+                       lambda: ci.attention_rows(q3, kc, vc, base, short, win, 0.09), 4 * b * win * G * D, 0, 0)
+
+
 FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12        # fp32 pipe at the highest SM clock
 
 
 @torch.no_grad()
-def bench_kernels(s, T=4096, B=8, context=4096):
+def bench_kernels(s, T=4096, B=8, context=4096, cases=kernel_cases):
     from ..ops.bench_kernels import _PEAKS, timed
     rows = []
-    for name, phase, fn, nbytes, flop, fp32 in kernel_cases(s, T, B, context):
+    for name, phase, fn, nbytes, flop, fp32 in cases(s, T, B, context):
         us = timed(fn) * 1e3
         bounds = {"hbm": nbytes / (_PEAKS["hbm_gbs"] * 1e3), "tensor": flop / (_PEAKS["bf16_tflops"] * 1e6),
                   "fp32": fp32 / (FP32_TFLOPS * 1e6)}
@@ -203,13 +323,13 @@ def bench_kernels(s, T=4096, B=8, context=4096):
     return rows, _PEAKS["source"]
 
 
-def main(sizes, kernels=True, iters=20, clocks=None):
+def main(sizes, kernels=True, iters=20, clocks=None, model="pafodra"):
     """One JSON line per size; ``clocks``: a sampler with start() / stop() run around each model's timings."""
     from ..ops import cuda as cu
     cu.lib()
     for name in sizes:
         s = SIZES[name]
-        for which in ("pafodra", "llama"):
+        for which in ("pafodra", "llama") if model == "pafodra" else ("megozen", "pafodra attention"):
             if clocks is not None:
                 sampler = clocks()
                 sampler.start()
@@ -221,7 +341,7 @@ def main(sizes, kernels=True, iters=20, clocks=None):
             print(json.dumps(out), flush=True)
         cu.check_err_flag()
         if kernels:
-            rows, source = bench_kernels(s)
+            rows, source = bench_kernels(s, cases=kernel_cases if model == "pafodra" else megozen_cases)
             print(json.dumps({"size": name, "peaks": source, "kernels": rows}), flush=True)
             cu.check_err_flag()
     return 0

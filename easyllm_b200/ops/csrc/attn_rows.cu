@@ -12,6 +12,7 @@
 //
 // Latent attention (one key row shared by all query heads, whose first dv columns are also the value, bf16) has a
 // kernel of its own, attn_latent_kernel: the products run on mma.sync m16n8k16 over a key tile that is read once.
+#include "sm100.cuh"
 #include "vec.cuh"
 
 namespace ell {
@@ -29,6 +30,7 @@ struct AttnRowsArgs {
   int window;                     // keys a row sees at most (INT_MAX: all)
   const void* gate;               // [n, ldg] of the activation type, or null
   int ldg;
+  int* err;                       // error word (latent kernel)
 };
 
 // Keys row t sees: the last min(len, window) of its rows.
@@ -270,37 +272,72 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
   }
 }
 
-// One CTA per (row, head): merge the ranges' triples.  Empty ranges carry max = -inf, sum = 0.
+// One CTA per (row, head): merge the ranges' triples.  Empty ranges carry max = -inf, sum = 0.  The ranges' weights are
+// formed once (a range a thread), then every thread sums its columns over the ranges with independent loads.
+constexpr int kArMaxSplits = 64;
 template <typename T>
 __global__ void __launch_bounds__(kArThreads) attn_rows_merge_kernel(const AttnRowsArgs a) {
-  const int t = blockIdx.x, h = blockIdx.y;
-  const float* pt = a.part + ((size_t)t * a.H + h) * a.splits * (a.dv + 2);
+  __shared__ float weight[kArMaxSplits];
+  const int t = blockIdx.x, h = blockIdx.y, step = a.dv + 2;
+  const float* pt = a.part + ((size_t)t * a.H + h) * a.splits * step;
   const int used = min(a.splits, (row_keys(a, t).len + a.range - 1) / a.range);
-  const float gate = row_gate<T>(a, t, h);
-  float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
-  for (int s = 0; s < used; ++s) m = fmaxf(m, pt[(size_t)s * (a.dv + 2)]);
-  float den = a.sink != nullptr ? expf(a.sink[h] - m) : 0.f;
-  for (int s = 0; s < used; ++s) den += pt[(size_t)s * (a.dv + 2) + 1] * expf(pt[(size_t)s * (a.dv + 2)] - m);
-  for (int c = threadIdx.x; c < a.dv; c += kArThreads) {
-    float o = 0.f;
-    for (int s = 0; s < used; ++s) o = fmaf(pt[(size_t)s * (a.dv + 2) + 2 + c], expf(pt[(size_t)s * (a.dv + 2)] - m), o);
-    reinterpret_cast<T*>(a.out)[((size_t)t * a.H + h) * a.dv + c] = from_f<T>(o / den * gate);
+  if (threadIdx.x < 32) {
+    const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
+    const float m0 = s0 < used ? pt[(size_t)s0 * step] : -INFINITY, m1 = s1 < used ? pt[(size_t)s1 * step] : -INFINITY;
+    const float l0 = s0 < used ? pt[(size_t)s0 * step + 1] : 0.f, l1 = s1 < used ? pt[(size_t)s1 * step + 1] : 0.f;
+    const float sk = a.sink != nullptr ? a.sink[h] : -INFINITY;
+    const float m = fmaxf(warp_max(fmaxf(m0, m1)), sk);            // finite: the first range has a key
+    const float e0 = expf(m0 - m), e1 = expf(m1 - m);
+    const float den = warp_sum(l0 * e0 + l1 * e1) + (a.sink != nullptr ? expf(sk - m) : 0.f);
+    const float f = row_gate<T>(a, t, h) / den;
+    weight[s0] = e0 * f;
+    weight[s1] = e1 * f;
+  }
+  __syncthreads();
+  T* out = reinterpret_cast<T*>(a.out) + ((size_t)t * a.H + h) * a.dv;
+  if (a.dv % 2 == 0) {                                             // triples start at even places
+    for (int c = threadIdx.x * 2; c < a.dv; c += 2 * kArThreads) {
+      float2 o = make_float2(0.f, 0.f);
+#pragma unroll 8
+      for (int s = 0; s < used; ++s) {
+        const float2 v = *reinterpret_cast<const float2*>(pt + (size_t)s * step + 2 + c);
+        o.x = fmaf(v.x, weight[s], o.x);
+        o.y = fmaf(v.y, weight[s], o.y);
+      }
+      out[c] = from_f<T>(o.x);
+      out[c + 1] = from_f<T>(o.y);
+    }
+  } else {
+    for (int c = threadIdx.x; c < a.dv; c += kArThreads) {
+      float o = 0.f;
+#pragma unroll 8
+      for (int s = 0; s < used; ++s) o = fmaf(pt[(size_t)s * step + 2 + c], weight[s], o);
+      out[c] = from_f<T>(o);
+    }
   }
 }
 
 // ---- latent attention: all heads share one key row, its first dv columns are the value ---------------
-// A CTA of 8 warps takes (row t, 16 * MT query heads, a range of keys).  Tiles of 64 key rows come through two
-// shared-memory stages (cp.async); row strides are an odd number of 16-byte pieces, so ldmatrix meets no bank conflicts.
-//   scores   MT = 1: warp w multiplies keys 8 w .. 8 w + 7;  MT = 2: warps 0-3 take the first 16 heads, 4-7 the second,
-//            16 keys each.  Scores go to shared memory in fp32.
-//   softmax  a warp owns 2 * MT heads; two keys a lane; fp32 weights, their sum unrounded, the operand of P·V in bf16
-//   values   warp w owns columns [w, w + 1) * dv / 8 of all heads; the value operand is the key tile itself (ldmatrix
+// A CTA of 16 warps takes (row t, 16 * MT query heads, a range of keys).  Tiles of 64 key rows come through two
+// shared-memory stages as TMA boxes of 64 columns (128-byte swizzle: ldmatrix meets no bank conflicts).
+//   scores   a warp multiplies 16 heads with 32 keys over one of 8 / MT slices of the columns (k-steps of 16); the
+//            slices' sums go to shared memory in fp32
+//   softmax  a warp owns MT heads, 32 / MT lanes each; fp32 weights, their sum unrounded, the operand of P·V in bf16
+//   values   warp w owns columns [w, w + 1) * dv / 16 of all heads; the value operand is the key tile itself (ldmatrix
 //            with transposition); its rescaled accumulators stay in registers
-constexpr int kAlWarps = 8, kAlKeys = 64, kAlPStride = kAlKeys + 8, kAlSStride = kAlKeys + 4, kAlMaxNt = 8;
+constexpr int kAlWarps = 16, kAlKeys = 64, kAlPStride = kAlKeys + 8, kAlSStride = kAlKeys + 4, kAlMaxNt = 4;
+constexpr int kAlSRows = 8 * 16;                 // slices of the score product x heads
+constexpr int kAlErr = 14;
 
-__host__ __device__ inline int al_krow(int d) { return (d + 15) / 16 * 16 + 8; }
+constexpr int kAlBoxBytes = kAlKeys * 128;             // [64 keys x 64 columns]
+__host__ __device__ inline int al_krow(int d) { return (d + 15) / 16 * 16 + 8; }       // stride of a query row
 static int al_bytes(int d, int MT) {
-  return (2 * kAlKeys + 16 * MT) * al_krow(d) * 2 + 16 * MT * (kAlPStride * 2 + kAlSStride * 4 + 16);
+  return 1024 + 2 * ((d + 63) / 64) * kAlBoxBytes + 16 * MT * (al_krow(d) * 2 + kAlPStride * 2 + 16) +
+         kAlSRows * kAlSStride * 4 + 32;
+}
+// Place of a 16-byte piece (8 columns) of a key row in a stage.
+__device__ __forceinline__ uint32_t al_place(int row, int piece) {
+  return (uint32_t)((piece >> 3) * kAlBoxBytes + row * 128 + (((piece & 7) ^ (row & 7)) << 4));
 }
 
 __device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
@@ -319,39 +356,45 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
 }
 
 template <int MT>
-__global__ void __launch_bounds__(kAlWarps * 32) attn_latent_kernel(const AttnRowsArgs a) {
-  extern __shared__ __align__(16) uint8_t alsm[];
+__global__ void __launch_bounds__(kAlWarps * 32)
+attn_latent_kernel(const __grid_constant__ CUtensorMap tmK, const AttnRowsArgs a) {
+  extern __shared__ uint8_t alsm_raw[];
+  uint8_t* kv = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(alsm_raw) + 1023) & ~(uintptr_t)1023);
   constexpr int HM = 16 * MT;
-  const int krow = al_krow(a.d), dp = krow - 8;
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(alsm);
-  __nv_bfloat16* kv = qs + HM * krow;
-  __nv_bfloat16* ps = kv + 2 * kAlKeys * krow;
+  const int krow = al_krow(a.d), dp = krow - 8, boxes = (a.d + 63) / 64, stage_bytes = boxes * kAlBoxBytes;
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(kv + 2 * stage_bytes);
+  __nv_bfloat16* ps = qs + HM * krow;
   float* ss = reinterpret_cast<float*>(ps + HM * kAlPStride);
-  float* stat = ss + HM * kAlSStride;                  // max | sum | rescale, HM each
+  float* stat = ss + kAlSRows * kAlSStride;                  // max | sum | rescale, HM each
+  uint64_t* full = reinterpret_cast<uint64_t*>(stat + 4 * HM);      // one barrier a stage
+  int* gave_up = reinterpret_cast<int*>(full + 2);
   const int t = blockIdx.x, h0 = blockIdx.y * HM, nh = min(HM, a.H - h0), split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const RowKeys rk = row_keys(a, t);
   const int k0 = split * a.range, k1 = min(k0 + a.range, rk.len);
-  const __nv_bfloat16* kb = reinterpret_cast<const __nv_bfloat16*>(a.k) + rk.base * a.ldk;
   const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(a.q) + (size_t)t * a.ldq + (size_t)h0 * a.d;
   const int pieces = a.d / 8, padded = dp / 8;         // 16-byte pieces of a row
-  // rows and columns that the copies leave out read as zero
+  const int tail = k1 > k0 ? (k1 - k0 - 1) % kAlKeys + 1 : kAlKeys, tiles = k1 > k0 ? (k1 - k0 + kAlKeys - 1) / kAlKeys : 0;
+  // one thread: columns past d and rows past the tensor are zero-filled
+  auto load_tile = [&](int kt, int buf) {
+    sm100::mbar_expect_tx(&full[buf], (uint32_t)stage_bytes);
+    for (int c = 0; c < boxes; ++c)
+      sm100::tma_load_2d(kv + buf * stage_bytes + c * kAlBoxBytes, &tmK, &full[buf], c * 64, (int)rk.base + kt);
+  };
+  if (threadIdx.x == 0) {
+    sm100::mbar_init(&full[0], 1);
+    sm100::mbar_init(&full[1], 1);
+    *gave_up = *(volatile int*)a.err;                  // an earlier kernel already failed: do not wait on anything
+    sm100::fence_barrier_init();
+    if (tiles > 0 && *gave_up == 0) load_tile(k0, 0);  // on its way while the queries come
+  }
+  // query rows and columns past the end read as zero
   for (int i = threadIdx.x; i < HM * padded; i += kAlWarps * 32) {
     const int h = i / padded, c = i % padded;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (h < nh && c < pieces) v = *reinterpret_cast<const uint4*>(qb + (size_t)h * a.d + c * 8);
     *reinterpret_cast<uint4*>(qs + h * krow + c * 8) = v;
   }
-  auto load_tile = [&](int kt, int buf) {
-    __nv_bfloat16* dst = kv + buf * kAlKeys * krow;
-    const int cnt = min(kAlKeys, k1 - kt);
-    for (int i = threadIdx.x; i < kAlKeys * padded; i += kAlWarps * 32) {
-      const int r = i / padded, c = i % padded;
-      if (r < cnt && c < pieces) cp_async16(dst + r * krow + c * 8, kb + (size_t)(kt + r) * a.ldk + c * 8);
-      else *reinterpret_cast<uint4*>(dst + r * krow + c * 8) = make_uint4(0, 0, 0, 0);
-    }
-    cp_async_commit();
-  };
   if (threadIdx.x < HM) {
     stat[threadIdx.x] = -INFINITY;
     stat[HM + threadIdx.x] = 0.f;
@@ -368,76 +411,93 @@ __global__ void __launch_bounds__(kAlWarps * 32) attn_latent_kernel(const AttnRo
       for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
   const int g = lane >> 2, tq = lane & 3;
   const int l8 = lane & 7, quad = lane >> 3;
-  if (k0 < k1) load_tile(k0, 0);
-  int buf = 0;
-  for (int kt = k0; kt < k1; kt += kAlKeys, buf ^= 1) {
-    if (kt + kAlKeys < k1) {
-      load_tile(kt + kAlKeys, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
+  __syncthreads();
+  const bool dead = *gave_up != 0;
+  constexpr int KS = 8 / MT;                             // column slices of the score product
+  const int mt = MT == 1 ? 0 : warp >> 3, key0 = (warp & 1) * 32, slice = (warp >> 1) % KS;
+  for (int it = 0; it < tiles && !dead; ++it) {
+    const int buf = it & 1, kt = k0 + it * kAlKeys;
+    uint8_t* ks = kv + buf * stage_bytes;
+    if (threadIdx.x == 0 && it + 1 < tiles) load_tile(kt + kAlKeys, buf ^ 1);   // the end of the last step freed that stage
+    if (!sm100::mbar_wait(&full[buf], (it >> 1) & 1, gave_up)) *(volatile int*)gave_up = 1;
+    else if (it == tiles - 1)                            // rows past the range are other keys: their weight is 0, not their value
+      for (int i = threadIdx.x; i < (kAlKeys - tail) * padded; i += kAlWarps * 32)
+        *reinterpret_cast<uint4*>(ks + al_place(tail + i / padded, i % padded)) = make_uint4(0, 0, 0, 0);
     __syncthreads();
-    const __nv_bfloat16* ks = kv + buf * kAlKeys * krow;
-    // scores of 16 heads and MT * 8 keys
+    if (*(volatile int*)gave_up) {
+      if (threadIdx.x == 0) {
+        atomicCAS(a.err, 0, kAlErr);
+        const unsigned long long t0 = sm100::globaltimer_ns();          // copies still in flight land before the CTA ends
+        while (sm100::globaltimer_ns() - t0 < 200000ull) {
+        }
+      }
+      __syncthreads();
+      break;                                             // uniform: every thread reads the flag after the barrier
+    }
+    // scores of 16 heads and 32 keys over this warp's slice of the columns
     {
-      const int mt = MT == 1 ? 0 : warp >> 2, key0 = MT == 1 ? warp * 8 : (warp & 3) * 16;
-      float sc[MT][4];
+      float sc[4][4];
 #pragma unroll
-      for (int n = 0; n < MT; ++n)
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int i = 0; i < 4; ++i) sc[n][i] = 0.f;
       const __nv_bfloat16* qrow = qs + (mt * 16 + (quad & 1) * 8 + l8) * krow + (quad >> 1) * 8;
-      // 32 columns of 8 keys (MT 1), or 16 columns of 16 keys (MT 2), per ldmatrix
-      const __nv_bfloat16* krow_p = MT == 1 ? ks + (key0 + l8) * krow + quad * 8
-                                            : ks + (key0 + (quad >> 1) * 8 + l8) * krow + (quad & 1) * 8;
-      if (MT == 1) {
-        int c = 0;
-#pragma unroll 4
-        for (; c + 32 <= dp; c += 32) {
-          uint32_t a0[4], a1[4], b[4];
-          ldsm4(a0, qrow + c);
-          ldsm4(a1, qrow + c + 16);
-          ldsm4(b, krow_p + c);
-          mma_bf16(sc[0], a0, b[0], b[1]);
-          mma_bf16(sc[0], a1, b[2], b[3]);
-        }
-        if (c < dp) {                                    // a last single k-step: the lanes past it repeat its columns
-          uint32_t a0[4], b[4];
-          ldsm4(a0, qrow + c);
-          ldsm4(b, ks + (key0 + l8) * krow + c + (quad & 1) * 8);
-          mma_bf16(sc[0], a0, b[0], b[1]);
-        }
-      } else {
-#pragma unroll 4
-        for (int c = 0; c < dp; c += 16) {
-          uint32_t a0[4], b[4];
-          ldsm4(a0, qrow + c);
-          ldsm4(b, krow_p + c);
-          mma_bf16(sc[0], a0, b[0], b[1]);
-          mma_bf16(sc[MT - 1], a0, b[2], b[3]);
+      const int krow_i = key0 + (quad >> 1) * 8 + l8;
+#pragma unroll 3
+      for (int c = slice * 16; c < dp; c += KS * 16) {
+        uint32_t a0[4], b0[4], b1[4];
+        ldsm4(a0, qrow + c);
+        const uint32_t at = al_place(krow_i, (c >> 3) + (quad & 1));       // 16 rows on: the same swizzle
+        ldsm4(b0, ks + at);
+        ldsm4(b1, ks + at + 16 * 128);
+        mma_bf16(sc[0], a0, b0[0], b0[1]);
+        mma_bf16(sc[1], a0, b0[2], b0[3]);
+        mma_bf16(sc[2], a0, b1[0], b1[1]);
+        mma_bf16(sc[3], a0, b1[2], b1[3]);
+      }
+      float* dst = ss + (slice * HM + mt * 16 + g) * kAlSStride + key0 + tq * 2;
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        *reinterpret_cast<float2*>(dst + n * 8) = make_float2(sc[n][0], sc[n][1]);
+        *reinterpret_cast<float2*>(dst + 8 * kAlSStride + n * 8) = make_float2(sc[n][2], sc[n][3]);
+      }
+    }
+    __syncthreads();
+    {
+      constexpr int LH = 32 / MT, KL = kAlKeys / LH;       // lanes a head, keys a lane
+      const int hh = warp * MT + lane / LH, key = (lane % LH) * KL;
+      float sv[KL], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < KL; ++j) sv[j] = 0.f;
+#pragma unroll
+      for (int y = 0; y < KS; ++y) {
+        const float* row = ss + (y * HM + hh) * kAlSStride + key;
+#pragma unroll
+        for (int j = 0; j < KL; j += 2) {
+          const float2 v = *reinterpret_cast<const float2*>(row + j);
+          sv[j] += v.x;
+          sv[j + 1] += v.y;
         }
       }
 #pragma unroll
-      for (int n = 0; n < MT; ++n)
+      for (int j = 0; j < KL; ++j) {
+        sv[j] = kt + key + j < k1 ? sv[j] * a.scale : -INFINITY;
+        mx = fmaxf(mx, sv[j]);
+      }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int key = key0 + n * 8 + tq * 2 + (i & 1), hh = mt * 16 + g + (i >> 1) * 8;
-          ss[hh * kAlSStride + key] = kt + key < k1 ? sc[n][i] * a.scale : -INFINITY;
-        }
-    }
-    __syncthreads();
+      for (int o = LH / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_old = stat[hh], m = fmaxf(m_old, mx);  // finite: the tile has a key
 #pragma unroll
-    for (int x = 0; x < 2 * MT; ++x) {
-      const int hh = warp * 2 * MT + x;
-      const float s0 = ss[hh * kAlSStride + lane], s1 = ss[hh * kAlSStride + 32 + lane];
-      const float m_old = stat[hh], m = fmaxf(m_old, warp_max(fmaxf(s0, s1)));     // finite: the tile has a key
-      const float e0 = expf(s0 - m), e1 = expf(s1 - m);
-      ps[hh * kAlPStride + lane] = __float2bfloat16_rn(e0);
-      ps[hh * kAlPStride + 32 + lane] = __float2bfloat16_rn(e1);
-      const float sum = warp_sum(e0 + e1);
-      __syncwarp();
-      if (lane == 0) {
+      for (int j = 0; j < KL; ++j) {
+        sv[j] = expf(sv[j] - m);
+        sum += sv[j];
+      }
+#pragma unroll
+      for (int j = 0; j < KL; j += 2)
+        *reinterpret_cast<__nv_bfloat162*>(ps + hh * kAlPStride + key + j) = __floats2bfloat162_rn(sv[j], sv[j + 1]);
+#pragma unroll
+      for (int o = LH / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if (lane % LH == 0) {                                // its lanes have read the old maximum: the shuffles above
         const float al = expf(m_old - m);
         stat[hh] = m;
         stat[HM + hh] = stat[HM + hh] * al + sum;
@@ -466,7 +526,7 @@ __global__ void __launch_bounds__(kAlWarps * 32) attn_latent_kernel(const AttnRo
 #pragma unroll
         for (int k = 0; k < kAlKeys / 32; ++k) {         // 32 keys x 8 columns per ldmatrix
           uint32_t b[4];
-          ldsm4_t(b, ks + (k * 32 + quad * 8 + l8) * krow + col0 + n * 8);
+          ldsm4_t(b, ks + al_place(k * 32 + quad * 8 + l8, col0 / 8 + n));
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             mma_bf16(acc[m][n], pa[m][2 * k], b[0], b[1]);
@@ -513,12 +573,18 @@ static int attn_latent_splits(int n, int H, int max_len) {
   long long s = kNumSMs / ctas;
   const long long most = (max_len + kAlKeys - 1) / kAlKeys;
   if (s > most) s = most;
-  if (s > 64) s = 64;
+  if (s > kArMaxSplits) s = kArMaxSplits;
   return s < 1 ? 1 : (int)s;
 }
 
+int make_tmap_bf16_2d(CUtensorMap* map, const void* ptr, uint64_t inner, uint64_t outer, uint64_t row_stride_bytes,
+                      uint32_t box_inner, uint32_t box_outer);
+
 template <int MT>
-static int launch_attn_latent(const AttnRowsArgs& a, cudaStream_t stream) {
+static int launch_attn_latent(const AttnRowsArgs& a, long long rows, cudaStream_t stream) {
+  CUtensorMap tk;
+  const int rc = make_tmap_bf16_2d(&tk, a.k, (uint64_t)a.d, (uint64_t)rows, (uint64_t)a.ldk * 2, 64, kAlKeys);
+  if (rc) return rc;
   const int bytes = al_bytes(a.d, MT);
   static int configured = 0;
   if (bytes > configured) {
@@ -526,14 +592,14 @@ static int launch_attn_latent(const AttnRowsArgs& a, cudaStream_t stream) {
     if (e != cudaSuccess) return (int)e;
     configured = bytes;
   }
-  attn_latent_kernel<MT><<<dim3(a.n, (a.H + 16 * MT - 1) / (16 * MT), a.splits), kAlWarps * 32, bytes, stream>>>(a);
+  attn_latent_kernel<MT><<<dim3(a.n, (a.H + 16 * MT - 1) / (16 * MT), a.splits), kAlWarps * 32, bytes, stream>>>(tk, a);
   if (a.splits > 1) attn_rows_merge_kernel<__nv_bfloat16><<<dim3(a.n, a.H), kArThreads, 0, stream>>>(a);
   return launch_status();
 }
 
 // Shapes of the mma kernel; everything else runs on attn_rows_kernel.
-static bool attn_latent_fits(int d, int dv, int ldq, int ldk, int H) {
-  return d % 8 == 0 && dv % 8 == 0 && dv <= d && dv <= 8 * kAlWarps * kAlMaxNt && ldq % 8 == 0 && ldk % 8 == 0 &&
+static bool attn_latent_fits(const void* k, int d, int dv, int ldq, int ldk, int H) {
+  return aligned_to(k, 16) && d % 8 == 0 && dv % 8 == 0 && dv <= d && dv <= 8 * kAlWarps * kAlMaxNt && ldq % 8 == 0 && ldk % 8 == 0 &&
          H <= 65535 && al_bytes(d, al_mt(H)) <= 227 * 1024;
 }
 
@@ -547,7 +613,7 @@ static int attn_rows_splits(int n, int H, int G, int max_len) {
   long long s = (4LL * kNumSMs + ctas - 1) / ctas;
   const long long most = (max_len + 255) / 256;
   if (s > most) s = most;
-  if (s > 64) s = 64;
+  if (s > kArMaxSplits) s = kArMaxSplits;
   return s < 1 ? 1 : (int)s;
 }
 
@@ -593,7 +659,7 @@ ELL_API int ell_attn_rows(const void* q, const void* k, const void* v, void* out
   if (H % G || dv > 8 * kArThreads || H > 65535) return -2;
   if (window <= 0) window = 0x7fffffff;
   if (max_len > window) max_len = window;
-  AttnRowsArgs a{q, k, v, out, part, base, len, sink, slopes, n, H, G, d, dv, ldq, ldk, ldv, 1, 0, scale, window, gate, ldg};
+  AttnRowsArgs a{q, k, v, out, part, base, len, sink, slopes, n, H, G, d, dv, ldq, ldk, ldv, 1, 0, scale, window, gate, ldg, nullptr};
   a.splits = attn_rows_splits(n, H, G, max_len);
   a.range = ((max_len + a.splits - 1) / a.splits + 63) / 64 * 64;
   if (a.splits > 1 && part == nullptr) return -2;
@@ -608,28 +674,28 @@ ELL_API int ell_attn_rows(const void* q, const void* k, const void* v, void* out
   return per == 4 ? launch_attn_rows<float, 4>(a, grid, vec, stream) : launch_attn_rows<float, 8>(a, grid, vec, stream);
 }
 
-// Latent attention: q [n, H, d] (rows of ldq), one key row [d] per position (rows of ldk) whose first dv columns are the
-// value -> out [n, H, dv].  bf16 shapes the mma kernel takes run there, others on attn_rows.
-ELL_API long long ell_attn_latent_scratch(int n, int H, int d, int dv, int ldq, int ldk, int max_len, int window, int is_bf16) {
+// Latent attention: q [n, H, d] (rows of ldq), one key row [d] per position (`rows` rows of ldk) whose first dv columns are
+// the value -> out [n, H, dv].  bf16 shapes the mma kernel takes run there, others on attn_rows.
+ELL_API long long ell_attn_latent_scratch(const void* k, int n, int H, int d, int dv, int ldq, int ldk, int max_len, int window, int is_bf16) {
   if (window > 0 && max_len > window) max_len = window;
-  if (!(is_bf16 && attn_latent_fits(d, dv, ldq, ldk, H))) return ell_attn_rows_scratch(n, H, 1, dv, max_len);
+  if (!(is_bf16 && attn_latent_fits(k, d, dv, ldq, ldk, H))) return ell_attn_rows_scratch(n, H, 1, dv, max_len);
   const int s = attn_latent_splits(n, H, max_len);
   return s == 1 ? 0 : (long long)n * H * s * (dv + 2);
 }
 
 ELL_API int ell_attn_latent(const void* q, const void* k, void* out, float* part, const int* base, const int* len,
                             const void* gate, int n, int H, int d, int dv, int ldq, int ldk, int ldg, int max_len, int window,
-                            float scale, int is_bf16, cudaStream_t stream) {
+                            long long rows, float scale, int is_bf16, int* err, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (!(is_bf16 && attn_latent_fits(d, dv, ldq, ldk, H)))
+  if (!(is_bf16 && attn_latent_fits(k, d, dv, ldq, ldk, H)))
     return ell_attn_rows(q, k, k, out, part, base, len, nullptr, nullptr, gate, n, H, 1, d, dv, ldq, ldk, ldk, ldg, max_len,
                          window, scale, is_bf16, stream);
-  if (!aligned_to(q, 16) || !aligned_to(k, 16) || !aligned_to(out, 16)) return -2;
+  if (!aligned_to(q, 16) || !aligned_to(k, 16) || !aligned_to(out, 16) || rows > 0x7fffffff) return -2;
   if (window <= 0) window = 0x7fffffff;
   if (max_len > window) max_len = window;
-  AttnRowsArgs a{q, k, k, out, part, base, len, nullptr, nullptr, n, H, 1, d, dv, ldq, ldk, ldk, 1, 0, scale, window, gate, ldg};
+  AttnRowsArgs a{q, k, k, out, part, base, len, nullptr, nullptr, n, H, 1, d, dv, ldq, ldk, ldk, 1, 0, scale, window, gate, ldg, err};
   a.splits = attn_latent_splits(n, H, max_len);
   a.range = ((max_len + a.splits - 1) / a.splits + kAlKeys - 1) / kAlKeys * kAlKeys;
   if (a.splits > 1 && part == nullptr) return -2;
-  return al_mt(H) == 1 ? launch_attn_latent<1>(a, stream) : launch_attn_latent<2>(a, stream);
+  return al_mt(H) == 1 ? launch_attn_latent<1>(a, rows, stream) : launch_attn_latent<2>(a, rows, stream);
 }

@@ -356,43 +356,67 @@ layer_norms_kernel(const float* __restrict__ x, const float* __restrict__ w1, co
 //   rotated query parts -> z, or, with q_dst, to q_dst [n, H, q_stride]: neighbouring dimensions 2i, 2i+1 are a pair,
 //     turned by the angle tables cos / sin [position, pairs]; dimensions past 2 * pairs pass unchanged
 //   latent -> divided by its root mean square, times norm_w;  key part -> rotated
-// Latent and key part also go to cache row base[t] + len[t] - 1 (rows of ldc), if there is a cache.  One CTA per token.
+// Latent and key part also go to cache row base[t] + len[t] - 1 (rows of ldc), if there is a cache.
+// One CTA per token; small enough that a dozen share an SM, since a token is a chain of dependent loads (its position,
+// the angles there) around few bytes.
+constexpr int kLatThreads = 128;
 template <typename T, int V>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kLatThreads, 12)
 latent_inputs_kernel(T* __restrict__ z, T* __restrict__ q_dst, T* __restrict__ cache, const float* __restrict__ norm_w,
                      const float* __restrict__ cosT, const float* __restrict__ sinT, const int* __restrict__ pos,
                      const int* __restrict__ base, const int* __restrict__ len, int H, int dim, int rot, int rank, int pairs,
                      int ldz, int q_stride, int ldc, float eps) {
-  __shared__ float red[8];
+  __shared__ float red[kLatThreads / 32];
   const int t = blockIdx.x;
   constexpr int VL = V == 8 ? 8 : 1;                    // pieces of the latent (any rank)
   T* row = z + (size_t)t * ldz;
-  const float* ct = cosT + (size_t)pos[t] * pairs;
-  const float* st = sinT + (size_t)pos[t] * pairs;
-  auto turn = [&](const T* src, T* dst, int c) {        // V consecutive dimensions from c on (V even)
-    float f[V];
-    load_v<V>(src + c, f);
+  const int place = pos[t], qw = dim + rot;
+  T* lat = row + (size_t)H * qw;
+  T* kr = lat + rank;
+  // the first piece of every thread stays in registers over the reduction
+  float first[VL], ss = 0.f;
+  const int c0 = threadIdx.x * VL;
+  if (c0 < rank) load_v<VL>(lat + c0, first);
+  else
 #pragma unroll
-    for (int j = 0; j < V / 2; ++j) {
-      const int i = c / 2 + j;
-      if (i < pairs) {
-        const float u = f[2 * j], v = f[2 * j + 1], cs = ct[i], sn = st[i];
-        f[2 * j] = u * cs - v * sn;
-        f[2 * j + 1] = v * cs + u * sn;
+    for (int j = 0; j < VL; ++j) first[j] = 0.f;
+  T* crow = cache != nullptr ? cache + ((size_t)base[t] + len[t] - 1) * ldc : nullptr;
+  // V consecutive dimensions from c on of the H query parts, then of the key part
+  const int per = rot / V;
+  for (int i = threadIdx.x; i < (H + 1) * per; i += kLatThreads) {
+    const int h = i / per, c = (i - h * per) * V;
+    const bool key = h == H;
+    float f[V];
+    load_v<V>((key ? kr : row + (size_t)h * qw + dim) + c, f);
+    if (c / 2 < pairs) {
+      const size_t at = (size_t)place * pairs + c / 2;
+      if (V == 8) {                                     // pairs is a multiple of 4
+        float cs[4], sn[4];
+        load_v<4>(cosT + at, cs);
+        load_v<4>(sinT + at, sn);
+#pragma unroll
+        for (int j = 0; j < V / 2; ++j) {
+          const float a = f[2 * j], b = f[2 * j + 1];
+          f[2 * j] = a * cs[j % 4] - b * sn[j % 4];
+          f[2 * j + 1] = b * cs[j % 4] + a * sn[j % 4];
+        }
+      } else {
+        const float a = f[0], b = f[1], cs = cosT[at], sn = sinT[at];
+        f[0] = a * cs - b * sn;
+        f[1] = b * cs + a * sn;
       }
     }
-    store_v<V>(dst + c, f);
-  };
-  const int per = rot / V, qw = dim + rot;
-  for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
-    const int h = i / per, c = (i % per) * V;
-    const T* src = row + (size_t)h * qw + dim;
-    turn(src, q_dst != nullptr ? q_dst + ((size_t)t * H + h) * q_stride : row + (size_t)h * qw + dim, c);
+    store_v<V>((key ? kr : q_dst != nullptr ? q_dst + ((size_t)t * H + h) * q_stride : row + (size_t)h * qw + dim) + c, f);
+    if (key && crow != nullptr) {
+      if (V == 8) store_v<V>(crow + rank + c, f);
+      else
+#pragma unroll
+        for (int j = 0; j < V; ++j) crow[rank + c + j] = from_f<T>(f[j]);
+    }
   }
-  T* lat = row + (size_t)H * qw;
-  T* crow = cache != nullptr ? cache + ((size_t)base[t] + len[t] - 1) * ldc : nullptr;
-  float ss = 0.f;
-  for (int c = threadIdx.x * VL; c < rank; c += blockDim.x * VL) {
+#pragma unroll
+  for (int j = 0; j < VL; ++j) ss = fmaf(first[j], first[j], ss);
+  for (int c = c0 + kLatThreads * VL; c < rank; c += kLatThreads * VL) {
     float f[VL];
     load_v<VL>(lat + c, f);
 #pragma unroll
@@ -402,24 +426,22 @@ latent_inputs_kernel(T* __restrict__ z, T* __restrict__ q_dst, T* __restrict__ c
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
   ss = 0.f;
-  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) ss += red[i];
+#pragma unroll
+  for (int i = 0; i < kLatThreads / 32; ++i) ss += red[i];
   const float r = 1.f / sqrtf(ss / rank + eps);
-  for (int c = threadIdx.x * VL; c < rank; c += blockDim.x * VL) {
+  for (int c = c0; c < rank; c += kLatThreads * VL) {
     float f[VL], w[VL];
-    load_v<VL>(lat + c, f);
+    if (c == c0) {
+#pragma unroll
+      for (int j = 0; j < VL; ++j) f[j] = first[j];
+    } else {
+      load_v<VL>(lat + c, f);
+    }
     load_v<VL>(norm_w + c, w);
 #pragma unroll
     for (int j = 0; j < VL; ++j) f[j] = f[j] * r * w[j];
     store_v<VL>(lat + c, f);
     if (crow != nullptr) store_v<VL>(crow + c, f);
-  }
-  T* kr = lat + rank;
-  for (int c = threadIdx.x * V; c < rot; c += blockDim.x * V) {
-    turn(kr, kr, c);
-    if (crow != nullptr) {
-#pragma unroll
-      for (int j = 0; j < V; ++j) crow[rank + c + j] = kr[c + j];
-    }
   }
 }
 
@@ -569,11 +591,11 @@ ELL_API int ell_latent_inputs(void* z, void* q_dst, void* cache, const float* no
                               int pairs, int ldz, int q_stride, int ldc, float eps, int is_bf16, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (rot % 2 || 2 * pairs > rot || rank < 1) return -2;
-  const bool v = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && ldz % 8 == 0 && q_stride % 8 == 0 && ldc % 8 == 0 &&
+  const bool v = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && pairs % 4 == 0 && aligned_to(cosT, 16) && aligned_to(sinT, 16) && ldz % 8 == 0 && q_stride % 8 == 0 && ldc % 8 == 0 &&
                  aligned_to(z, 16) && aligned_to(q_dst, 16) && aligned_to(cache, 16) && aligned_to(norm_w, 16);
 #define ELL_LAT(T, V)                                                                                                   \
-  latent_inputs_kernel<T, V><<<n, 256, 0, stream>>>((T*)z, (T*)q_dst, (T*)cache, norm_w, cosT, sinT, pos, base, len, H, \
-                                                    dim, rot, rank, pairs, ldz, q_stride, ldc, eps)
+  latent_inputs_kernel<T, V><<<n, kLatThreads, 0, stream>>>((T*)z, (T*)q_dst, (T*)cache, norm_w, cosT, sinT, pos, base, \
+                                                            len, H, dim, rot, rank, pairs, ldz, q_stride, ldc, eps)
   if (is_bf16) {
     if (v) ELL_LAT(__nv_bfloat16, 8);
     else ELL_LAT(__nv_bfloat16, 2);

@@ -266,11 +266,12 @@ def attention_latent(q, rows, dv, base, length, max_len, scale, window=None, gat
         raise ValueError("attention_latent: key rows of the queries' dtype and size")
     out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
     shape = (c_int(T), c_int(H), c_int(d), c_int(dv), c_int(_heads(q, "q")), c_int(ldk))
-    need = lib().ell_attn_latent_scratch(*shape, c_int(max_len), c_int(window or 0), _bf(q.dtype))
+    need = lib().ell_attn_latent_scratch(_p(rows), *shape, c_int(max_len), c_int(window or 0), _bf(q.dtype))
     part = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
     g, ldg = _gate(gate, q)
     _check(lib().ell_attn_latent(_p(q), _p(rows), _p(out), _p(part), _p(base), _p(length), g, *shape, ldg, c_int(max_len),
-                                 c_int(window or 0), c_float(scale), _bf(q.dtype), _stream()), "attn_latent", 2 if need else 1)
+                                 c_int(window or 0), c_longlong(rows.shape[0]), c_float(scale), _bf(q.dtype), _p(err_flag(q.device)), _stream()),
+           "attn_latent", 2 if need else 1)
     return out
 
 

@@ -5,7 +5,8 @@
 Cases: gemm_nt, gemm_nt_n4096, gemm_dgrad, gemm_wgrad, gemm_ag, gemm_rs, gemm_ar (single-CTA kernel), the same with
 the prefix gemm_pair_ (CTA-pair kernel) plus gemm_pair_agk (gather of the reduction rows into the weight-gradient
 GEMM) and gemm_pair_ce (LM head with the cross-entropy epilogue), flash_fwd, flash_bwd, rmsnorm_fwd, rmsnorm_bwd,
-swiglu, rope, adam, ce.
+swiglu, rope, adam, ce, attn_latent (decoding, 64 sequences of 4096 tokens, 32 heads over a latent of 512 + 64),
+flash_latent (one prompt of 4096 tokens, keys of 128 + 64, a window of 1024).
 Inputs are larger than L2 (126 MB) where the op is memory-bound but hold well under a few GB,
 so a full-section profiler capture of 1-3 launches ends by itself in a minute or two.
 """
@@ -105,6 +106,17 @@ def main():
         p = torch.randn(n, device="cuda"); g = torch.randn(n, device="cuda"); m = torch.zeros(n, device="cuda")
         v = torch.zeros(n, device="cuda"); low = torch.empty(n, **bf)
         fn = lambda: cu.adam(p, g, m, v, low, 1e-4, 0.9, 0.95, 1e-8, 0.1, 3)          # noqa: E731
+    elif c == "attn_latent":
+        from . import cuda_infer as ci
+        q = torch.randn(64, 32, 576, **bf); rows = torch.randn(64 * 4096, 576, **bf)
+        base = torch.arange(0, 64 * 4096, 4096, dtype=torch.int32, device="cuda")
+        ln = torch.full((64,), 4096, dtype=torch.int32, device="cuda")
+        fn = lambda: ci.attention_latent(q, rows, 512, base, ln, 4096, 0.07)          # noqa: E731
+    elif c == "flash_latent":
+        from . import cuda_infer as ci
+        z = torch.randn(4096, 32 * 192 + 576, **bf); kv = torch.randn(4096, 32 * 256, **bf)
+        rs = torch.zeros(4096, dtype=torch.int32, device="cuda")
+        fn = lambda: ci.attention_latent_prefill(z, kv, 32, 128, 64, 512, 128, rs, 0.07, 1024)   # noqa: E731
     elif c == "ce":
         lg = torch.randn(4096, 32000, **bf); t = torch.randint(0, 32000, (4096,), device="cuda")
         fn = lambda: cu.ce_fwd(lg, t, 0, 32000)                                       # noqa: E731

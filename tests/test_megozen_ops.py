@@ -86,7 +86,7 @@ def test_rotary_tables_follow_the_scaled_frequencies(r):
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("H,dim,rt,rank,dims", [(4, 32, 16, 48, 16), (3, 10, 6, 13, 4), (1, 5, 2, 7, 2), (16, 128, 64, 512, 64),
-                                                (2, 8, 24, 8, 16)])
+                                                (2, 8, 24, 8, 16), (5, 8, 64, 1200, 32)])
 @pytest.mark.parametrize("separate", [False, True])
 def test_rotations_latent_norm_and_cache_rows(device, dtype, H, dim, rt, rank, dims, separate):
     from easyllm_b200.models.layers import YarnRotaryTables
