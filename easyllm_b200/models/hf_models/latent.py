@@ -27,7 +27,7 @@ class LatentAttention(nn.Module):
         super().__init__()
         self.h, self.d, self.r, self.dv, self.rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
         self.scale, self.eps = float(m["scale"]), eps
-        self.window = m["mask"]["size"] if m.get("mask") else None
+        self.window = (m.get("mask") or {}).get("size")
         self.rotary = YarnRotaryTables(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
 
         def lin(i, o):

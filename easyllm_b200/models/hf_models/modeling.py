@@ -168,8 +168,9 @@ def _megozen_arch(cfg: dict) -> HFArch:
         dims = l.mixer["rot"]["dims"]
         if dims % 2 or l.mixer["rot_dim"] % 2 or not 0 < dims <= l.mixer["rot_dim"]:
             raise ValueError(f"layer {i}: {dims} rotated dimensions of {l.mixer['rot_dim']}")
-        if l.mixer.get("mask") and l.mixer["mask"]["size"] < 1:
-            raise ValueError(f"layer {i}: a window of {l.mixer['mask']['size']} tokens")
+        window = (l.mixer.get("mask") or {}).get("size")
+        if window is not None and window < 1:
+            raise ValueError(f"layer {i}: a window of {window} tokens")
     return HFArch(family="megozen", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layers=layers,
                   num_hidden_layers=len(layers), num_attention_heads=layers[0].mixer["heads"] if layers else 1,
                   num_key_value_heads=1, norm_eps=cfg["norm"]["eps"], block_norm="layer_norm", expert_form="glu",
