@@ -92,9 +92,12 @@ def _time(fn, iters):
 
 
 @torch.no_grad()
-def bench_model(which, s, prefills, decodes, context, iters):
+def bench_model(which, s, prefills, decodes, context, iters, sampler=None):
     from ..models.hf_models.state import DecodeGraph
     model = build(which, s)
+    torch.cuda.synchronize()
+    if sampler is not None:
+        sampler.start()
     rows = []
     gen = torch.Generator().manual_seed(1)
 
@@ -324,17 +327,16 @@ def bench_kernels(s, T=4096, B=8, context=4096, cases=kernel_cases):
 
 
 def main(sizes, kernels=True, iters=20, clocks=None, model="pafodra"):
-    """One JSON line per size; ``clocks``: a sampler with start() / stop() run around each model's timings."""
+    """One JSON line per size; ``clocks``: a sampler with start() / stop() run around each model's timings
+    (not around its making)."""
     from ..ops import cuda as cu
     cu.lib()
     for name in sizes:
         s = SIZES[name]
         for which in ("pafodra", "llama") if model == "pafodra" else ("megozen", "pafodra attention"):
-            if clocks is not None:
-                sampler = clocks()
-                sampler.start()
+            sampler = clocks() if clocks is not None else None
             l0 = cu.LAUNCHES
-            out = bench_model(which, s, [(1, 4096), (8, 512), (1, 512)], [1, 8, 64], 4096, iters)
+            out = bench_model(which, s, [(1, 4096), (8, 512), (1, 512)], [1, 8, 64], 4096, iters, sampler)
             out.update(size=name, shape=s, launches=cu.LAUNCHES - l0)
             if clocks is not None:
                 out["clocks"] = sampler.stop()
